@@ -10,7 +10,8 @@
 //                          kept in `state` [rows, taps - 1, C] (the last taps - 1 inputs; zeros before position 0).
 //   b200_silu_rows         x <- silu(x) in place on a column slice of fp32 rows (the activation of projections that enter a
 //                          scan without a convolution, done once instead of by every CTA that reads them).
-//   b200_short_conv_tail   advances that tail over the step's runs (launched after the convolution has read the old one).
+//   b200_short_conv_tail   advances that tail over the step's runs (launched after the convolution has read the old one); for
+//                          a decode batch the convolution does it itself. `in_bias`: a bias that belongs to the inputs.
 //   b200_delta_gates       q, k -> unit vectors per head (q also times `qscale`); a -> exp(-exp(A_log[h]) softplus(a + bias));
 //                          b -> sigmoid(b); in place, fp32.
 //   b200_linear_scan       per head, state S [D, Dv] (fp32, in `state` [rows, H, D, Dv]):
@@ -25,7 +26,7 @@
 //   b200_ssm_gates         step sizes of a selective state space: dt = softplus(x + bias), a = exp(-exp(A_log) dt), b = dt.
 //   b200_scan_readout      what follows a scan per token: optional division of each head by max(|last column|, e) + den_eps,
 //                          optional skip D_h x, optional silu gate BEFORE the norm, RMS norm over equal column groups,
-//                          weight (one per column, or shared by the groups), optional sigmoid gate AFTER the norm.
+//                          weight (one per column, or shared by the groups), optional sigmoid or silu gate AFTER the norm.
 //                          Columns of S are independent, so a thread owns R rows of one column, the lanes that share a
 //                          column reduce their partial dot products by shuffles, and a CTA owns a block of columns of one
 //                          (run, head): tokens are walked in order, staged through shared memory in chunks.
@@ -36,12 +37,23 @@ namespace b200 {
 
 __device__ __forceinline__ float silu_f(float v) { return v / (1.f + expf(-v)); }
 
+// V = 1 or 4 neighbouring elements as fp32 (V = 4: on a boundary of four elements)
+template <int V, typename T> __device__ __forceinline__ void load_f32(const T* p, float (&v)[V]) {
+  if (V == 4 && sizeof(T) == 4) *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(p);
+  else if (V == 4) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 a = unpack_bf16x2(raw.x), b = unpack_bf16x2(raw.y);
+    v[0] = a.x; v[V > 1 ? 1 : 0] = a.y; v[V > 2 ? 2 : 0] = b.x; v[V - 1] = b.y;
+  } else v[0] = to_f32<T>(p[0]);
+}
+
 // V channels per thread (V = 4: rows of x, y, the tail and C are multiples of four floats on 16-byte boundaries)
-template <int V, typename TY>
-__global__ void short_conv_kernel(const float* __restrict__ x, long long ldx, const float* __restrict__ w,
-                                  const float* __restrict__ bias, const float* __restrict__ state, const int* __restrict__ pos,
+// step_tail: every token is a run of its own, so the thread that reads a channel's old tail also advances it
+template <int V, typename TX, typename TY>
+__global__ void short_conv_kernel(const TX* __restrict__ x, long long ldx, const float* __restrict__ w,
+                                  const float* __restrict__ bias, float* __restrict__ state, const int* __restrict__ pos,
                                   const int* __restrict__ slot, TY* __restrict__ y, long long ldy, int tokens, int C, int taps,
-                                  int act, int residual) {
+                                  int act, int residual, int step_tail) {
   const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   const int CV = C / V;
   if (idx >= (long long)tokens * CV) return;
@@ -49,26 +61,39 @@ __global__ void short_conv_kernel(const float* __restrict__ x, long long ldx, co
   const int p = pos[t], s = slot[t];
   // nb: tokens of the same run right before t (at most taps - 1 matter)
   int nb = 0;
-  while (nb < taps - 1 && t - nb - 1 >= 0 && slot[t - nb - 1] == s) ++nb;
-  float acc[V], own[V];
+  if (!step_tail)
+    while (nb < taps - 1 && t - nb - 1 >= 0 && slot[t - nb - 1] == s) ++nb;
+  float acc[V], own[V], prev[V];
 #pragma unroll
-  for (int e = 0; e < V; ++e) { acc[e] = bias ? bias[c + e] : 0.f; own[e] = 0.f; }
+  for (int e = 0; e < V; ++e) { acc[e] = bias ? bias[c + e] : 0.f; own[e] = 0.f; prev[e] = 0.f; }
   for (int d = 0; d < taps; ++d) {                       // d tokens back
-    if (p - d < 0) break;
-    const float* src = d <= nb ? x + (long long)(t - d) * ldx + c : state + ((long long)s * (taps - 1) + (taps - 1 - (d - nb))) * C + c;
+    if (p - d < 0 && !step_tail) break;
     float v[V];
-    if (V == 4) *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(src);
-    else v[0] = src[0];
+    float* old = state + ((long long)s * (taps - 1) + (taps - 1 - (d - nb))) * C + c;      // read where d > nb
+    if (p - d < 0) {
+#pragma unroll
+      for (int e = 0; e < V; ++e) v[e] = 0.f;
+    } else if (d <= nb) {
+      load_f32<V, TX>(x + (long long)(t - d) * ldx + c, v);
+    } else {
+      load_f32<V, float>(old, v);
+    }
+    if (step_tail && d > 0) {                            // entry taps - 1 - d held the input d tokens back: it takes the next one
+#pragma unroll
+      for (int e = 0; e < V; ++e) old[e] = prev[e];
+    }
 #pragma unroll
     for (int e = 0; e < V; ++e) {
       acc[e] = fmaf(w[(long long)(c + e) * taps + (taps - 1 - d)], v[e], acc[e]);
       if (d == 0) own[e] = v[e];
+      prev[e] = v[e];
     }
   }
 #pragma unroll
   for (int e = 0; e < V; ++e) acc[e] = (act ? silu_f(acc[e]) : acc[e]) + (residual ? own[e] : 0.f);
   TY* dst = y + (long long)t * ldy + c;
   if (V == 4 && sizeof(TY) == 4) *reinterpret_cast<float4*>(dst) = *reinterpret_cast<const float4*>(acc);
+  else if (V == 4) *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16x2(acc[0], acc[1]), pack_bf16x2(acc[V - 2], acc[V - 1]));
   else {
 #pragma unroll
     for (int e = 0; e < V; ++e) dst[e] = from_f32<TY>(acc[e]);
@@ -93,7 +118,8 @@ __global__ void silu_rows_kernel(float* __restrict__ x, long long ld, long long 
   else px[0] = v[0];
 }
 
-__global__ void short_conv_tail_kernel(const float* __restrict__ x, long long ldx, float* __restrict__ state,
+template <typename TX>
+__global__ void short_conv_tail_kernel(const TX* __restrict__ x, long long ldx, const float* __restrict__ in_bias, float* __restrict__ state,
                                        const int* __restrict__ runs, const int* __restrict__ pos, const int* __restrict__ slot,
                                        int n_runs, int C, int taps) {
   const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -108,7 +134,7 @@ __global__ void short_conv_tail_kernel(const float* __restrict__ x, long long ld
   for (int i = 0; i < L; ++i) {
     const int q = p0 + n - L + i;                        // position whose input lands in entry i
     float v = 0.f;
-    if (q >= p0) v = x[(long long)(first + (q - p0)) * ldx + c];
+    if (q >= p0) v = to_f32<TX>(x[(long long)(first + (q - p0)) * ldx + c]) + (in_bias ? in_bias[c] : 0.f);
     else if (q >= 0) v = st[(long long)(q - p0 + L) * C];
     nv[i] = v;
   }
@@ -468,7 +494,7 @@ __global__ void __launch_bounds__(256)
 scan_readout_kernel(const float* __restrict__ o, int ocols, const float* __restrict__ e, float den_eps, float oscale,
                     const float* __restrict__ skip, const float* __restrict__ x, long long ldx,
                     const float* __restrict__ pre, long long ldpre, const float* __restrict__ post, long long ldpost,
-                    const float* __restrict__ w, int w_full, TO* __restrict__ out, int H, int Dv, int groups, float eps) {
+                    int post_silu, const float* __restrict__ w, int w_full, TO* __restrict__ out, int H, int Dv, int groups, float eps) {
   extern __shared__ float row[];                         // [N] + [groups]
   const long long t = blockIdx.x;
   const int N = H * Dv, GS = N / groups;
@@ -493,27 +519,36 @@ scan_readout_kernel(const float* __restrict__ o, int ocols, const float* __restr
   __syncthreads();
   for (int c = threadIdx.x; c < N; c += blockDim.x) {
     float v = row[c] * gsum[c / GS] * w[w_full ? c : c % GS];
-    if (post) v *= 1.f / (1.f + expf(-post[t * ldpost + c]));
+    if (post) { const float z = post[t * ldpost + c]; v *= (post_silu ? z : 1.f) / (1.f + expf(-z)); }
     out[t * N + c] = from_f32<TO>(v);
   }
 }
 }  // namespace b200
 
-B200_API int b200_short_conv_ex(const float* x, long long ldx, const float* w, const float* bias, const float* state,
+B200_API int b200_short_conv_ex(const void* x, long long ldx, const float* w, const float* bias, float* state,
                                 const int* pos, const int* slot, void* y, long long ldy, int tokens, int C, int taps, int act,
-                                int residual, int y_dtype, void* stream) {
+                                int residual, int step_tail, int x_dtype, int y_dtype, void* stream) {
   using namespace b200;
   if (tokens <= 0) return 0;
   if (C <= 0 || taps < 1 || taps > kMaxTaps) return B200_ERR_BAD_SHAPE;
-  if (y_dtype != B200_DT_FP32 && y_dtype != B200_DT_BF16) return B200_ERR_UNSUPPORTED;
+  if ((y_dtype != B200_DT_FP32 && y_dtype != B200_DT_BF16) || (x_dtype != B200_DT_FP32 && x_dtype != B200_DT_BF16))
+    return B200_ERR_UNSUPPORTED;
   cudaStream_t st = (cudaStream_t)stream;
-  const bool vec = C % 4 == 0 && ldx % 4 == 0 && ldy % 4 == 0 &&
-                   !((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(state)) & 15);
+  const bool vec = C % 4 == 0 && ldx % 4 == 0 && ldy % 4 == 0 && !(reinterpret_cast<uintptr_t>(state) & 15) &&
+                   !(reinterpret_cast<uintptr_t>(x) & (x_dtype == B200_DT_FP32 ? 15 : 7)) &&
+                   !(reinterpret_cast<uintptr_t>(y) & (y_dtype == B200_DT_FP32 ? 15 : 7));
   const long long n = (long long)tokens * (vec ? C / 4 : C);
   const unsigned grid = (unsigned)((n + 255) / 256);
-#define CONV(VV, TY) short_conv_kernel<VV, TY><<<grid, 256, 0, st>>>(x, ldx, w, bias, state, pos, slot, (TY*)y, ldy, tokens, C, taps, act, residual)
-  if (y_dtype == B200_DT_FP32) { if (vec) CONV(4, float); else CONV(1, float); }
-  else { if (vec) CONV(4, __nv_bfloat16); else CONV(1, __nv_bfloat16); }
+#define CONV(VV, TX, TY)                                                                                                     \
+  short_conv_kernel<VV, TX, TY><<<grid, 256, 0, st>>>((const TX*)x, ldx, w, bias, state, pos, slot, (TY*)y, ldy, tokens, C, taps, act, \
+                                                      residual, step_tail)
+#define CONV_X(TX)                                                                                                           \
+  do {                                                                                                                       \
+    if (y_dtype == B200_DT_FP32) { if (vec) CONV(4, TX, float); else CONV(1, TX, float); }                                   \
+    else { if (vec) CONV(4, TX, __nv_bfloat16); else CONV(1, TX, __nv_bfloat16); }                                           \
+  } while (0)
+  if (x_dtype == B200_DT_FP32) CONV_X(float); else CONV_X(__nv_bfloat16);
+#undef CONV_X
 #undef CONV
   B200_LAUNCH_CHECK();
   return 0;
@@ -521,7 +556,8 @@ B200_API int b200_short_conv_ex(const float* x, long long ldx, const float* w, c
 
 B200_API int b200_short_conv(const float* x, long long ldx, const float* w, const float* state, const int* pos, const int* slot,
                              float* y, long long ldy, int tokens, int C, int taps, int act, void* stream) {
-  return b200_short_conv_ex(x, ldx, w, nullptr, state, pos, slot, y, ldy, tokens, C, taps, act, 0, B200_DT_FP32, stream);
+  return b200_short_conv_ex(x, ldx, w, nullptr, const_cast<float*>(state), pos, slot, y, ldy, tokens, C, taps, act, 0, 0, B200_DT_FP32,
+                            B200_DT_FP32, stream);
 }
 
 B200_API int b200_silu_rows(float* x, long long ld, long long rows, int cols, void* stream) {
@@ -535,13 +571,19 @@ B200_API int b200_silu_rows(float* x, long long ld, long long rows, int cols, vo
   return 0;
 }
 
-B200_API int b200_short_conv_tail(const float* x, long long ldx, float* state, const int* runs, const int* pos, const int* slot,
-                                  int n_runs, int C, int taps, void* stream) {
+B200_API int b200_short_conv_tail(const void* x, long long ldx, const float* in_bias, float* state, const int* runs, const int* pos,
+                                  const int* slot, int n_runs, int C, int taps, int x_dtype, void* stream) {
   using namespace b200;
   if (n_runs <= 0 || taps <= 1) return 0;
   if (C <= 0 || taps > kMaxTaps) return B200_ERR_BAD_SHAPE;
   const long long n = (long long)n_runs * C;
-  short_conv_tail_kernel<<<(unsigned)((n + 255) / 256), 256, 0, (cudaStream_t)stream>>>(x, ldx, state, runs, pos, slot, n_runs, C, taps);
+  const unsigned grid = (unsigned)((n + 255) / 256);
+  cudaStream_t st = (cudaStream_t)stream;
+  if (x_dtype == B200_DT_FP32)
+    short_conv_tail_kernel<float><<<grid, 256, 0, st>>>((const float*)x, ldx, in_bias, state, runs, pos, slot, n_runs, C, taps);
+  else if (x_dtype == B200_DT_BF16)
+    short_conv_tail_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>((const __nv_bfloat16*)x, ldx, in_bias, state, runs, pos, slot, n_runs, C, taps);
+  else return B200_ERR_UNSUPPORTED;
   B200_LAUNCH_CHECK();
   return 0;
 }
@@ -637,7 +679,7 @@ B200_API int b200_ssm_gates(const float* dt, long long ld, const float* dt_bias,
 
 B200_API int b200_scan_readout(const float* o, int ocols, const float* e, float den_eps, float oscale, const float* skip,
                                const float* x, long long ldx, const float* pre, long long ldpre, const float* post,
-                               long long ldpost, const float* w, int w_full, void* out, long long tokens, int H, int Dv,
+                               long long ldpost, int post_silu, const float* w, int w_full, void* out, long long tokens, int H, int Dv,
                                int groups, float eps, int out_dtype, void* stream) {
   using namespace b200;
   if (tokens <= 0) return 0;
@@ -650,7 +692,7 @@ B200_API int b200_scan_readout(const float* o, int ocols, const float* e, float 
   do {                                                                                                                       \
     auto kern = scan_readout_kernel<TO>;                                                                                     \
     if (smem > 48 * 1024) B200_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));    \
-    kern<<<(unsigned)tokens, 256, smem, st>>>(o, ocols, e, den_eps, oscale, skip, x, ldx, pre, ldpre, post, ldpost, w, w_full,  \
+    kern<<<(unsigned)tokens, 256, smem, st>>>(o, ocols, e, den_eps, oscale, skip, x, ldx, pre, ldpre, post, ldpost, post_silu, w, w_full,  \
                                               (TO*)out, H, Dv, groups, eps);                                                 \
   } while (0)
   if (out_dtype == B200_DT_FP32) READOUT(float);

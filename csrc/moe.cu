@@ -10,8 +10,11 @@
 //                      they are or renormalised to sum 1. Rows of W_r past the experts are per-token gates: their sigmoid
 //                      goes to gate_out (the gate of a shared expert). One warp per token; ties go to the lower index.
 //   b200_moe_dispatch  the expert-sorted, tile-padded row layout of the assignments (a stable counting sort in one launch).
+//                      Expert indices past the last one (identity experts) get no row: dest -1.
+//   b200_moe_gather    the rows of that layout: xs[dest[r]] = h[tok[r]] (padding rows are left as they are).
 //   b200_moe_combine   out[t] = sum_k p[t, k] * y[dest[t * top + k]] (+ gate[t] * shared[t]) in fp32 (y: the expert-sorted
-//                      rows the grouped GEMM wrote), a fixed order of additions per token.
+//                      rows the grouped GEMM wrote), a fixed order of additions per token; an assignment without a row adds
+//                      p * ident[t] (the token's own fp32 row).
 #include "common.cuh"
 #include "../include/b200_ops.h"
 
@@ -229,7 +232,10 @@ moe_dispatch_kernel(const long long* __restrict__ top_i, long long* __restrict__
   }
   if (blockIdx.x != 0) return;
   for (int x = tid; x < E; x += blockDim.x) counts[x] = cnt[x];
-  for (int r = tid; r < R; r += blockDim.x) tok[r] = r / top;
+  for (int r = tid; r < R; r += blockDim.x) {
+    tok[r] = r / top;
+    if (ids[r] == (unsigned short)0xffff) dest[r] = -1;            // no expert with weights: no row
+  }
   for (int t = tid; t < n_tiles; t += blockDim.x) {
     const int row = t * tile;
     int lo = 0, hi = E;                                            // the last expert whose segment starts at or before row
@@ -243,18 +249,59 @@ moe_dispatch_kernel(const long long* __restrict__ top_i, long long* __restrict__
   }
 }
 
-template <typename T>
+// xs[dest[r]] = h[tok[r]], rows of `chunks` 16-byte (or, for rows that are not whole chunks, 2-byte) units; one warp per row
+template <typename U>
+__global__ void __launch_bounds__(256)
+moe_gather_kernel(const U* __restrict__ h, const long long* __restrict__ dest, const long long* __restrict__ tok, U* __restrict__ xs,
+                  long long R, int chunks) {
+  const long long r = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (r >= R) return;
+  const long long d = dest[r];
+  if (d < 0) return;
+  const U* src = h + tok[r] * chunks;
+  U* dst = xs + d * chunks;
+  for (int c = threadIdx.x & 31; c < chunks; c += 32) dst[c] = src[c];
+}
+
+template <int V, typename T> __device__ __forceinline__ void combine_load(const T* p, float (&v)[V]) {
+  if (V == 4 && sizeof(T) == 4) *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(p);
+  else if (V == 4) {
+    T raw[4];
+    *reinterpret_cast<uint2*>(raw) = *reinterpret_cast<const uint2*>(p);
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] = to_f32<T>(raw[e]);
+  } else v[0] = to_f32<T>(p[0]);
+}
+
+// V neighbouring columns per thread (4 where the width allows)
+template <typename T, int V>
 __global__ void moe_combine_kernel(const T* __restrict__ y, const long long* __restrict__ dest, const float* __restrict__ p,
-                                   const T* __restrict__ shared, const float* __restrict__ gate, float* __restrict__ out,
-                                   long long tokens, int W, int top) {
-  const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+                                   const T* __restrict__ shared, const float* __restrict__ gate, const float* __restrict__ ident,
+                                   float* __restrict__ out, long long tokens, int W, int top) {
+  const long long idx = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * V;
   if (idx >= tokens * W) return;
   const long long t = idx / W;
   const int c = (int)(idx - t * W);
-  float a = 0.f;
-  for (int k = 0; k < top; ++k) a = fmaf(p[t * top + k], to_f32<T>(y[dest[t * top + k] * W + c]), a);
-  if (shared) a = fmaf(gate ? gate[t] : 1.f, to_f32<T>(shared[idx]), a);
-  out[idx] = a;
+  float a[V], v[V];
+#pragma unroll
+  for (int e = 0; e < V; ++e) a[e] = 0.f;
+  for (int k = 0; k < top; ++k) {
+    const long long d = dest[t * top + k];
+    const float w = p[t * top + k];
+    if (d >= 0) combine_load<V, T>(y + d * W + c, v);
+    else if (ident) combine_load<V, float>(ident + idx, v);
+    else continue;
+#pragma unroll
+    for (int e = 0; e < V; ++e) a[e] = fmaf(w, v[e], a[e]);
+  }
+  if (shared) {
+    const float w = gate ? gate[t] : 1.f;
+    combine_load<V, T>(shared + idx, v);
+#pragma unroll
+    for (int e = 0; e < V; ++e) a[e] = fmaf(w, v[e], a[e]);
+  }
+  if (V == 4) *reinterpret_cast<float4*>(out + idx) = *reinterpret_cast<const float4*>(a);
+  else out[idx] = a[0];
 }
 
 }  // namespace b200
@@ -323,18 +370,39 @@ B200_API int b200_moe_dispatch(const long long* top_i, long long* dest, long lon
   return 0;
 }
 
+B200_API int b200_moe_gather(const void* h, const long long* dest, const long long* tok, void* xs, long long assignments,
+                             long long row_bytes, void* stream) {
+  if (assignments <= 0) return 0;
+  if (row_bytes <= 0 || row_bytes % 2 || row_bytes / 2 > 0x7fffffffLL) return B200_ERR_BAD_SHAPE;
+  cudaStream_t st = (cudaStream_t)stream;
+  const unsigned grid = (unsigned)((assignments + 7) / 8);
+  if (row_bytes % 16 == 0 && !((reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(xs)) & 15))
+    moe_gather_kernel<uint4><<<grid, 256, 0, st>>>((const uint4*)h, dest, tok, (uint4*)xs, assignments, (int)(row_bytes / 16));
+  else
+    moe_gather_kernel<unsigned short><<<grid, 256, 0, st>>>((const unsigned short*)h, dest, tok, (unsigned short*)xs, assignments, (int)(row_bytes / 2));
+  B200_LAUNCH_CHECK();
+  return 0;
+}
+
 B200_API int b200_moe_combine(const void* y, const long long* dest, const float* p, const void* shared, const float* gate,
-                              float* out, long long tokens, int W, int top, int dtype, void* stream) {
+                              const float* ident, float* out, long long tokens, int W, int top, int dtype, void* stream) {
   cudaStream_t st = (cudaStream_t)stream;
   if (tokens <= 0) return 0;
-  const unsigned grid = (unsigned)((tokens * W + 255) / 256);
-  if (dtype == B200_DT_BF16)
-    moe_combine_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>((const __nv_bfloat16*)y, dest, p, (const __nv_bfloat16*)shared, gate, out, tokens, W, top);
-  else if (dtype == B200_DT_FP16)
-    moe_combine_kernel<__half><<<grid, 256, 0, st>>>((const __half*)y, dest, p, (const __half*)shared, gate, out, tokens, W, top);
-  else if (dtype == B200_DT_FP32)
-    moe_combine_kernel<float><<<grid, 256, 0, st>>>((const float*)y, dest, p, (const float*)shared, gate, out, tokens, W, top);
+  auto al = [](const void* q, int n) { return !(reinterpret_cast<uintptr_t>(q) & (n - 1)); };
+  const int es = dtype == B200_DT_FP32 ? 16 : 8;
+  const bool vec = W % 4 == 0 && al(y, es) && (!shared || al(shared, es)) && (!ident || al(ident, 16)) && al(out, 16);
+  const long long n = tokens * W / (vec ? 4 : 1);
+  const unsigned grid = (unsigned)((n + 255) / 256);
+#define CB(T)                                                                                                                \
+  do {                                                                                                                       \
+    if (vec) moe_combine_kernel<T, 4><<<grid, 256, 0, st>>>((const T*)y, dest, p, (const T*)shared, gate, ident, out, tokens, W, top); \
+    else moe_combine_kernel<T, 1><<<grid, 256, 0, st>>>((const T*)y, dest, p, (const T*)shared, gate, ident, out, tokens, W, top);     \
+  } while (0)
+  if (dtype == B200_DT_BF16) CB(__nv_bfloat16);
+  else if (dtype == B200_DT_FP16) CB(__half);
+  else if (dtype == B200_DT_FP32) CB(float);
   else return B200_ERR_UNSUPPORTED;
+#undef CB
   B200_LAUNCH_CHECK();
   return 0;
 }

@@ -7,10 +7,13 @@
 //   window <= 0 means every j <= p.
 //   a_m = softmax_j(scale q_{h,m} . k_{g,m,j}) V_g        g = h / (H / G)
 //   M = 2, combine:  o = a_0 - lambda a_1 ;  o <- o / sqrt(mean(o^2) + eps) * post      (differential attention)
-//   otherwise:       o = a_0 (M = 1)
+//   otherwise:       o = a_0 post (M = 1)
 //
 // b200_qknorm_rope_store   per-(head, map) RMS norm with a weight over D, rotary on the first `rot` dims in the split layout
 //                          (dim i pairs with i + rot/2), q -> q_out in the cache dtype, k and v -> their pages.
+// b200_conv_qknorm_store   what stands in front of one-map attention whose projections pass a short causal convolution: bias,
+//                          convolution over time on every channel of q | k | v (inputs before the run come from a carried tail),
+//                          per-row RMS norm without a weight (v optional), q times a factor that grows with the position.
 // b200_multimap_attn       per-token attention in fp32 arithmetic over a 16-bit or 32-bit cache; prompt pieces and decoded
 //                          tokens take the same path: a vector kernel (16-byte row chunks, the heads of a KV group share the
 //                          K/V reads, `nsplit` key ranges + a merge kernel for few tokens with many keys) and a scalar one
@@ -79,6 +82,123 @@ qknorm_rope_store_kernel(const float* __restrict__ proj, long long ld, const flo
   }
 }
 
+// proj [tokens, ld] = q (H rows of D) | k (G rows of D) | v (G rows of Dv). A warp owns one of these rows over TB consecutive
+// tokens, every lane up to VI pairs (V = 2) or single channels; the last taps - 1 inputs of a channel stay in registers from
+// token to token and are fetched anew (from proj, the tail, or zeros) where a run starts inside the block.
+// TAPS: the convolution's taps at compile time.
+constexpr int kConvMaxTaps = 5;
+template <typename TX, typename T, int TAPS, int V, int VI>
+__global__ void __launch_bounds__(128)
+conv_qknorm_store_kernel(const TX* __restrict__ proj, long long ld, const float* __restrict__ bias, const float* __restrict__ w,
+                         const float* __restrict__ tail, const int* __restrict__ pos, const int* __restrict__ slot,
+                         const int* __restrict__ table, int max_blocks, T* __restrict__ q_out, T* __restrict__ ck, T* __restrict__ cv,
+                         int tokens, int H, int G, int D, int Dv, int block_size, float eps, float temp_coef, float temp_every,
+                         int norm_qk, int norm_v, int TB) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int r = blockIdx.y * 4 + warp;
+  if (r >= H + 2 * G) return;
+  const bool is_v = r >= H + G;
+  const int RS = is_v ? Dv : D;
+  const int col0 = is_v ? (H + G) * D + (r - H - G) * Dv : r * D;
+  const int C = (H + G) * D + G * Dv;
+  constexpr int L = TAPS - 1;
+  float wt[VI][V][TAPS], hist[VI][V][L > 0 ? L : 1], b[VI][V];
+#pragma unroll
+  for (int i = 0; i < VI; ++i)
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      const int c = (lane + 32 * i) * V + e;
+      b[i][e] = (bias && c < RS) ? bias[col0 + c] : 0.f;
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) wt[i][e][j] = c < RS ? w[(long long)(col0 + c) * TAPS + j] : 0.f;
+#pragma unroll
+      for (int j = 0; j < L; ++j) hist[i][e][j] = 0.f;
+    }
+  auto load = [&](int t, int i, float (&v)[V]) {           // the biased inputs of token t
+    const int c = (lane + 32 * i) * V;
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] = 0.f;
+    if (c < RS) {
+      const TX* p = proj + (long long)t * ld + col0 + c;
+      if (V == 2 && sizeof(TX) == 2) {
+        const float2 f = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(p));
+        v[0] = f.x; v[V - 1] = f.y;
+      } else if (V == 2) {
+        const float2 f = *reinterpret_cast<const float2*>(p);
+        v[0] = f.x; v[V - 1] = f.y;
+      } else v[0] = to_f32<TX>(p[0]);
+#pragma unroll
+      for (int e = 0; e < V; ++e) v[e] += b[i][e];
+    }
+  };
+  const int t0 = blockIdx.x * TB, t1 = min(tokens, t0 + TB);
+  int ps = -1, pp = -2;
+  for (int t = t0; t < t1; ++t) {
+    const int p = pos[t], s = slot[t];
+    if (L > 0 && !(s == ps && p == pp + 1)) {              // not the token after the last one: fetch what lies before it
+      int nb = 0;
+      while (nb < L && t - nb - 1 >= 0 && slot[t - nb - 1] == s && pos[t - nb - 1] == p - nb - 1) ++nb;
+#pragma unroll
+      for (int d = 1; d <= L; ++d)                         // d tokens back -> hist[L - d]
+#pragma unroll
+        for (int i = 0; i < VI; ++i) {
+          float v[V];
+#pragma unroll
+          for (int e = 0; e < V; ++e) v[e] = 0.f;
+          if (p - d >= 0) {
+            if (d <= nb) load(t - d, i, v);
+            else {
+#pragma unroll
+              for (int e = 0; e < V; ++e) {
+                const int c = (lane + 32 * i) * V + e;
+                if (c < RS) v[e] = tail[((long long)s * L + (L - (d - nb))) * C + col0 + c];
+              }
+            }
+          }
+#pragma unroll
+          for (int e = 0; e < V; ++e) hist[i][e][L > 0 ? L - d : 0] = v[e];
+        }
+    }
+    ps = s; pp = p;
+    float y[VI][V], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < VI; ++i) {
+      float v[V];
+      load(t, i, v);
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        float a = 0.f;
+#pragma unroll
+        for (int j = 0; j < L; ++j) a = fmaf(wt[i][e][j], hist[i][e][j], a);
+        a = fmaf(wt[i][e][TAPS - 1], v[e], a);
+#pragma unroll
+        for (int j = 0; j + 1 < L; ++j) hist[i][e][j] = hist[i][e][j + 1];
+        if (L > 0) hist[i][e][L > 0 ? L - 1 : 0] = v[e];
+        y[i][e] = a;
+        ss = fmaf(a, a, ss);
+      }
+    }
+    float f = 1.f;
+    if (is_v ? norm_v : norm_qk) f = rsqrtf(warp_sum(ss) / RS + eps);
+    if (r < H && temp_coef != 0.f) f *= 1.f + temp_coef * logf((float)floor((double)(p + 1) / (double)temp_every) + 1.f);
+    T* dst;
+    if (r < H) dst = q_out + ((long long)t * H + r) * D;
+    else {
+      const long long blk = table[(long long)s * max_blocks + p / block_size];
+      const int off = p % block_size;
+      dst = is_v ? cv + ((blk * G + (r - H - G)) * block_size + off) * Dv : ck + ((blk * G + (r - H)) * block_size + off) * D;
+    }
+#pragma unroll
+    for (int i = 0; i < VI; ++i) {
+      const int c = (lane + 32 * i) * V;
+      if (c >= RS) continue;
+      if (V == 2 && sizeof(T) == 2) *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16x2(y[i][0] * f, y[i][V - 1] * f);
+      else if (V == 2) *reinterpret_cast<float2*>(dst + c) = make_float2(y[i][0] * f, y[i][V - 1] * f);
+      else dst[c] = from_f32<T>(y[i][0] * f);
+    }
+  }
+}
+
 constexpr int kMaxDv = 256;
 constexpr int kAcc = kMaxDv / 32;
 constexpr int kMaxMaps = 2;
@@ -112,7 +232,7 @@ __device__ __forceinline__ float dot_qk<__nv_bfloat16>(const float* __restrict__
 template <typename T>
 __global__ void __launch_bounds__(128)
 multimap_attn_kernel(const T* __restrict__ q, const T* __restrict__ ck, const T* __restrict__ cv, const int* __restrict__ pos,
-                     const int* __restrict__ slot, const int* __restrict__ table, int max_blocks, T* __restrict__ out, int tokens,
+                     const int* __restrict__ slot, const int* __restrict__ table, int max_blocks, T* __restrict__ out, long long ldo, int tokens,
                      int H, int G, int M, int D, int Dv, int block_size, float scale, int window, int keep_first, int combine,
                      float lambda, float post, float eps) {
   extern __shared__ float qs[];                          // [warps, D]
@@ -177,7 +297,7 @@ multimap_attn_kernel(const T* __restrict__ q, const T* __restrict__ ck, const T*
 #pragma unroll
     for (int a = 0; a < kAcc; ++a) res[a] = fmaf(coef, acc[a] * inv, res[a]);
   }
-  float mult = 1.f;
+  float mult = post;
   if (combine) {
     float ss = 0.f;
 #pragma unroll
@@ -185,7 +305,7 @@ multimap_attn_kernel(const T* __restrict__ q, const T* __restrict__ ck, const T*
     ss = warp_sum(ss);
     mult = rsqrtf(ss / Dv + eps) * post;
   }
-  T* orow = out + ((long long)t * H + h) * Dv;
+  T* orow = out + (long long)t * ldo + (long long)h * Dv;
 #pragma unroll
   for (int a = 0; a < kAcc; ++a) {
     const int d = lane + 32 * a;
@@ -204,9 +324,9 @@ multimap_attn_kernel(const T* __restrict__ q, const T* __restrict__ ck, const T*
 template <typename T, int HB, int VC>
 __global__ void __launch_bounds__(128, 4)               // four CTAs per SM: a decode batch of 64 x 4 groups x 2 maps is one wave
 multimap_attn_vec_kernel(const T* __restrict__ q, const T* __restrict__ ck, const T* __restrict__ cv, const int* __restrict__ pos,
-                         const int* __restrict__ slot, const int* __restrict__ table, int max_blocks, T* __restrict__ out,
+                         const int* __restrict__ slot, const int* __restrict__ table, int max_blocks, T* __restrict__ out, long long ldo,
                          float* __restrict__ part, int H, int G, int M, int D, int Dv, int bs_log2, float scale, int window,
-                         int keep_first, int nsplit, int CP, int CPK, int CPV) {
+                         int keep_first, int nsplit, float post, int CP, int CPK, int CPV) {
   constexpr int E = 16 / sizeof(T);
   extern __shared__ float sm[];                          // [4 warps][HB][Dv + 2]
   const int t = blockIdx.x;
@@ -370,7 +490,7 @@ multimap_attn_vec_kernel(const T* __restrict__ q, const T* __restrict__ ck, cons
       }
     }
     if (direct) {
-      out[((long long)t * H + h) * Dv + d] = from_f32<T>(lt > 0.f ? at / lt : 0.f);
+      out[(long long)t * ldo + (long long)h * Dv + d] = from_f32<T>(lt > 0.f ? at / lt * post : 0.f);
     } else {
       float* pr = part + ((((long long)t * H + h) * M + m) * nsplit + split) * LDW;
       if (d == 0) { pr[0] = mt; pr[1] = lt; }
@@ -382,7 +502,7 @@ multimap_attn_vec_kernel(const T* __restrict__ q, const T* __restrict__ ck, cons
 // one warp per (token, head): merges the key ranges of every map, then the combination and the norm
 template <typename T>
 __global__ void __launch_bounds__(128)
-multimap_attn_merge_kernel(const float* __restrict__ part, T* __restrict__ out, long long items, int M, int Dv, int nsplit,
+multimap_attn_merge_kernel(const float* __restrict__ part, T* __restrict__ out, long long ldo, int H, long long items, int M, int Dv, int nsplit,
                            int combine, float lambda, float post, float eps) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long long item = (long long)blockIdx.x * 4 + warp;            // (token, head)
@@ -414,7 +534,7 @@ multimap_attn_merge_kernel(const float* __restrict__ part, T* __restrict__ out, 
 #pragma unroll
     for (int a = 0; a < kAcc; ++a) res[a] = fmaf(coef, at[a] * inv, res[a]);
   }
-  float mult = 1.f;
+  float mult = post;
   if (combine) {
     float ss = 0.f;
 #pragma unroll
@@ -425,7 +545,7 @@ multimap_attn_merge_kernel(const float* __restrict__ part, T* __restrict__ out, 
 #pragma unroll
   for (int a = 0; a < kAcc; ++a) {
     const int d = lane + 32 * a;
-    if (d < Dv) out[item * Dv + d] = from_f32<T>(res[a] * mult);
+    if (d < Dv) out[item / H * ldo + item % H * Dv + d] = from_f32<T>(res[a] * mult);
   }
 }
 }  // namespace b200
@@ -446,8 +566,47 @@ B200_API int b200_qknorm_rope_store(const float* proj, long long ld, const float
   return 0;
 }
 
+B200_API int b200_conv_qknorm_store(const void* proj, long long ld, const float* bias, const float* w, const float* tail, const int* pos,
+                                    const int* slot, const int* table, int max_blocks, void* q_out, void* ck, void* cv, int tokens,
+                                    int H, int G, int D, int Dv, int taps, int block_size, float eps, float temp_coef,
+                                    float temp_every, int norm_qk, int norm_v, int x_dtype, int dtype, void* stream) {
+  using namespace b200;
+  if (tokens <= 0) return 0;
+  if (H <= 0 || G <= 0 || D <= 0 || Dv <= 0 || block_size <= 0 || taps < 1 || !(temp_every > 0.f)) return B200_ERR_BAD_SHAPE;
+  const int big = D > Dv ? D : Dv;
+  if (taps > kConvMaxTaps || big > 512) return B200_ERR_TOO_LARGE;
+  const int es = x_dtype == B200_DT_FP32 ? 4 : 2, eo = dtype == B200_DT_FP32 ? 4 : 2;
+  auto al = [](const void* p_, int n) { return !(reinterpret_cast<uintptr_t>(p_) & (n - 1)); };
+  const bool v2 = D % 2 == 0 && Dv % 2 == 0 && ld % 2 == 0 && al(proj, 2 * es) && al(q_out, 2 * eo) && al(ck, 2 * eo) && al(cv, 2 * eo);
+  const int TB = tokens <= 512 ? 1 : 8;
+  dim3 grid((tokens + TB - 1) / TB, (H + 2 * G + 3) / 4);
+  cudaStream_t st = (cudaStream_t)stream;
+#define CQ(TX, T, TAPSV, VV, VIV)                                                                                              \
+  conv_qknorm_store_kernel<TX, T, TAPSV, VV, VIV><<<grid, 128, 0, st>>>((const TX*)proj, ld, bias, w, tail, pos, slot, table,   \
+      max_blocks, (T*)q_out, (T*)ck, (T*)cv, tokens, H, G, D, Dv, block_size, eps, temp_coef, temp_every, norm_qk, norm_v, TB)
+#define CQ_V(TX, T, TAPSV)                                                                                                     \
+  do {                                                                                                                         \
+    if (v2 && big <= 64) CQ(TX, T, TAPSV, 2, 1); else if (v2 && big <= 128) CQ(TX, T, TAPSV, 2, 2);                             \
+    else if (v2 && big <= 256) CQ(TX, T, TAPSV, 2, 4); else if (v2) CQ(TX, T, TAPSV, 2, 8);                                    \
+    else if (big <= 128) CQ(TX, T, TAPSV, 1, 4); else CQ(TX, T, TAPSV, 1, 16);                                                 \
+  } while (0)
+#define CQ_T(TX, T)                                                                                                            \
+  switch (taps) {                                                                                                              \
+    case 1: CQ_V(TX, T, 1); break; case 2: CQ_V(TX, T, 2); break; case 3: CQ_V(TX, T, 3); break; case 4: CQ_V(TX, T, 4); break; \
+    default: CQ_V(TX, T, 5); break;                                                                                            \
+  }
+  if (x_dtype == B200_DT_BF16 && dtype == B200_DT_BF16) { CQ_T(__nv_bfloat16, __nv_bfloat16) }
+  else if (x_dtype == B200_DT_FP32 && dtype == B200_DT_FP32) { CQ_T(float, float) }
+  else return B200_ERR_UNSUPPORTED;
+#undef CQ_T
+#undef CQ_V
+#undef CQ
+  B200_LAUNCH_CHECK();
+  return 0;
+}
+
 B200_API int b200_multimap_attn(const void* q, const void* ck, const void* cv, const int* pos, const int* slot, const int* table,
-                                int max_blocks, void* out, float* part, int tokens, int H, int G, int M, int D, int Dv,
+                                int max_blocks, void* out, long long ldo, float* part, int tokens, int H, int G, int M, int D, int Dv,
                                 int block_size, float scale, int window, int keep_first, int nsplit, int combine, float lambda,
                                 float post, float eps, int dtype, void* stream) {
   using namespace b200;
@@ -478,7 +637,7 @@ B200_API int b200_multimap_attn(const void* q, const void* ck, const void* cv, c
       const size_t smem = (size_t)4 * HB * (Dv + 2) * sizeof(float);
 #define MMV2(T, HBV, VCV)                                                                                                    \
   multimap_attn_vec_kernel<T, HBV, VCV><<<grid, 128, smem, st>>>((const T*)q, (const T*)ck, (const T*)cv, pos, slot, table,   \
-      max_blocks, (T*)out, part, H, G, M, D, Dv, bs_log2, scale, window, keep_first, nsplit, CP, CPK, CPV)
+      max_blocks, (T*)out, ldo, part, H, G, M, D, Dv, bs_log2, scale, window, keep_first, nsplit, post, CP, CPK, CPV)
 #define MMV(T, HBV)                                                                                                          \
   do { if (VC == 2) MMV2(T, HBV, 2); else MMV2(T, HBV, 1); } while (0)
 #define MMV_T(T)                                                                                                             \
@@ -486,7 +645,7 @@ B200_API int b200_multimap_attn(const void* q, const void* ck, const void* cv, c
     if (HB == 4) MMV(T, 4); else if (HB == 2) MMV(T, 2); else MMV(T, 1);                                                     \
     if (!direct)                                                                                                             \
       multimap_attn_merge_kernel<T><<<(unsigned)(((long long)tokens * H + 3) / 4), 128, 0, st>>>(                             \
-          part, (T*)out, (long long)tokens * H, M, Dv, nsplit, combine, lambda, post, eps);                                  \
+          part, (T*)out, ldo, H, (long long)tokens * H, M, Dv, nsplit, combine, lambda, post, eps);                                  \
   } while (0)
       if (dtype == B200_DT_BF16) MMV_T(__nv_bfloat16);
       else if (dtype == B200_DT_FP16) MMV_T(__half);
@@ -504,7 +663,7 @@ B200_API int b200_multimap_attn(const void* q, const void* ck, const void* cv, c
   if (smem > 48 * 1024) return B200_ERR_TOO_LARGE;
   const unsigned grid = (unsigned)(((long long)tokens * H + nw - 1) / nw);
   B200_DISPATCH_T(dtype, multimap_attn_kernel<T><<<grid, nw * 32, smem, st>>>(
-      (const T*)q, (const T*)ck, (const T*)cv, pos, slot, table, max_blocks, (T*)out, tokens, H, G, M, D, Dv, block_size, scale,
+      (const T*)q, (const T*)ck, (const T*)cv, pos, slot, table, max_blocks, (T*)out, ldo, tokens, H, G, M, D, Dv, block_size, scale,
       window, keep_first, combine, lambda, post, eps));
   B200_LAUNCH_CHECK();
   return 0;

@@ -6,7 +6,7 @@
 // tile's first row up to the diagonal; blocks in between are never fetched — with S = Q K^T and P V on mma.sync.m16n8k16
 // (K [64, D] and V [64, Dv] pages gathered through the block table with double-buffered cp.async; P stays in registers as
 // the A operand). Scores, running maximum / sum and both accumulators are fp32. After the last map the combination
-// a_0 - lambda a_1, the RMS norm over Dv and the post factor are applied in registers and the row is written once.
+// a_0 - lambda a_1 and the RMS norm over Dv (if asked for) and the post factor are applied in registers and the row is written once.
 //
 // tcgen05 is not used: tiles are ragged (1 .. 64 rows at any position), D and Dv are independent multiples of 16, and the
 // mask has two disjoint key ranges per row; the like kernel of the single-map paged attention makes the same choice.
@@ -22,7 +22,7 @@ template <int DK, int DVK>
 __global__ void __launch_bounds__(128)
 multimap_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ ck,
                          const __nv_bfloat16* __restrict__ cv, const int* __restrict__ tiles, const int* __restrict__ table,
-                         int max_blocks, __nv_bfloat16* __restrict__ out, int H, int G, int M, int bs_log2, float scale,
+                         int max_blocks, __nv_bfloat16* __restrict__ out, long long ldo, int H, int G, int M, int bs_log2, float scale,
                          int window, int keep_first, int combine, float lambda, float post, float eps) {
   constexpr int D = 16 * DK, Dv = 16 * DVK;
   constexpr int LDK = D + 8, LDV = Dv + 8;
@@ -203,7 +203,7 @@ multimap_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
       res[n][3] = fmaf(o[n][3], i1, res[n][3]);
     }
   }
-  float f0 = 1.f, f1 = 1.f;
+  float f0 = post, f1 = post;
   if (combine) {
     float s0 = 0.f, s1 = 0.f;
 #pragma unroll
@@ -223,15 +223,15 @@ multimap_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
   for (int n = 0; n < 2 * DVK; ++n) {
     const int d = n * 8 + 2 * (lane & 3);
     if (ra < nrows)
-      *reinterpret_cast<uint32_t*>(out + ((long long)(row0 + ra) * H + h) * Dv + d) = pack_bf16x2(res[n][0] * f0, res[n][1] * f0);
+      *reinterpret_cast<uint32_t*>(out + (long long)(row0 + ra) * ldo + h * Dv + d) = pack_bf16x2(res[n][0] * f0, res[n][1] * f0);
     if (rb < nrows)
-      *reinterpret_cast<uint32_t*>(out + ((long long)(row0 + rb) * H + h) * Dv + d) = pack_bf16x2(res[n][2] * f1, res[n][3] * f1);
+      *reinterpret_cast<uint32_t*>(out + (long long)(row0 + rb) * ldo + h * Dv + d) = pack_bf16x2(res[n][2] * f1, res[n][3] * f1);
   }
 }
 
 template <int DK, int DVK>
 static int launch(const void* q, const void* ck, const void* cv, const int* tiles, int n_tiles, const int* table, int max_blocks,
-                  void* out, int H, int G, int M, int block_size, float scale, int window, int keep_first, int combine,
+                  void* out, long long ldo, int H, int G, int M, int block_size, float scale, int window, int keep_first, int combine,
                   float lambda, float post, float eps, cudaStream_t st) {
   constexpr int LDK = 16 * DK + 8, LDV = 16 * DVK + 8;
   const size_t smem = ((size_t)(kQ + 2 * kK) * LDK + (size_t)2 * kK * LDV) * sizeof(__nv_bfloat16);
@@ -241,7 +241,7 @@ static int launch(const void* q, const void* ck, const void* cv, const int* tile
   while ((1 << bs_log2) < block_size) ++bs_log2;
   if ((1 << bs_log2) != block_size) return B200_ERR_UNSUPPORTED;
   kern<<<dim3(n_tiles, H), 128, smem, st>>>((const __nv_bfloat16*)q, (const __nv_bfloat16*)ck, (const __nv_bfloat16*)cv, tiles, table,
-                                             max_blocks, (__nv_bfloat16*)out, H, G, M, bs_log2, scale, window, keep_first, combine,
+                                             max_blocks, (__nv_bfloat16*)out, ldo, H, G, M, bs_log2, scale, window, keep_first, combine,
                                              lambda, post, eps);
   B200_LAUNCH_CHECK();
   return 0;
@@ -249,17 +249,17 @@ static int launch(const void* q, const void* ck, const void* cv, const int* tile
 }  // namespace b200
 
 B200_API int b200_multimap_attn_mma(const void* q, const void* ck, const void* cv, const int* tiles, int n_tiles, const int* table,
-                                    int max_blocks, void* out, int H, int G, int M, int D, int Dv, int block_size, float scale,
+                                    int max_blocks, void* out, long long ldo, int H, int G, int M, int D, int Dv, int block_size, float scale,
                                     int window, int keep_first, int combine, float lambda, float post, float eps, int dtype,
                                     void* stream) {
   using namespace b200;
   if (n_tiles <= 0) return 0;
   if (dtype != B200_DT_BF16 || !(scale > 0.f) || M < 1 || M > 2 || (combine && M != 2)) return B200_ERR_UNSUPPORTED;
-  if (H <= 0 || G <= 0 || H % G || H > 65535) return B200_ERR_BAD_SHAPE;
+  if (H <= 0 || G <= 0 || H % G || H > 65535 || (ldo & 1) || (reinterpret_cast<uintptr_t>(out) & 3)) return B200_ERR_BAD_SHAPE;
   cudaStream_t st = (cudaStream_t)stream;
 #define MM(DKV, DVKV)                                                                                                       \
   if (D == 16 * DKV && Dv == 16 * DVKV)                                                                                     \
-    return launch<DKV, DVKV>(q, ck, cv, tiles, n_tiles, table, max_blocks, out, H, G, M, block_size, scale, window, keep_first, \
+    return launch<DKV, DVKV>(q, ck, cv, tiles, n_tiles, table, max_blocks, out, ldo, H, G, M, block_size, scale, window, keep_first, \
                              combine, lambda, post, eps, st);
 #define MMROW(DKV) MM(DKV, 2) MM(DKV, 4) MM(DKV, 6) MM(DKV, 8)
   MMROW(2) MMROW(3) MMROW(4) MMROW(6) MMROW(8)

@@ -500,6 +500,45 @@ static int sandwich_launch(const void* y, const void* w_post, const float* res_i
   B200_LAUNCH_CHECK();
   return 0;
 }
+// y = a N(z) + b N(z^2) + c N(z^3) + e per row, N(v) = v / sqrt(mean(v^2) + eps): three power sums in one pass over the row,
+// then a cubic in z per element. One CTA per row; V elements per load.
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+poly_norm_kernel(const T* __restrict__ z, const float* __restrict__ act, T* __restrict__ y, int cols, float eps) {
+  __shared__ float red[32];
+  const T* zr = z + (long long)blockIdx.x * cols;
+  T* yr = y + (long long)blockIdx.x * cols;
+  float s1 = 0.f, s2 = 0.f, s3 = 0.f;
+  for (int i = threadIdx.x * V; i < cols; i += blockDim.x * V) {
+    T raw[V];
+    if (V > 1) *reinterpret_cast<uint4*>(raw) = *reinterpret_cast<const uint4*>(zr + i);
+    else raw[0] = zr[i];
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      const float v = to_f32<T>(raw[e]), v2 = v * v, v4 = v2 * v2;
+      s1 += v2;
+      s2 += v4;
+      s3 = fmaf(v4, v2, s3);
+    }
+  }
+  s1 = block_sum(s1, red);
+  s2 = block_sum(s2, red);
+  s3 = block_sum(s3, red);
+  const float n = (float)cols;
+  const float a = act[0] / sqrtf(s1 / n + eps), b = act[1] / sqrtf(s2 / n + eps), c = act[2] / sqrtf(s3 / n + eps), d = act[3];
+  for (int i = threadIdx.x * V; i < cols; i += blockDim.x * V) {
+    T raw[V];
+    if (V > 1) *reinterpret_cast<uint4*>(raw) = *reinterpret_cast<const uint4*>(zr + i);
+    else raw[0] = zr[i];
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      const float v = to_f32<T>(raw[e]);
+      raw[e] = from_f32<T>(fmaf(v, fmaf(v, fmaf(v, c, b), a), d));
+    }
+    if (V > 1) *reinterpret_cast<uint4*>(yr + i) = *reinterpret_cast<const uint4*>(raw);
+    else yr[i] = raw[0];
+  }
+}
 }  // namespace b200
 
 B200_API int b200_sandwich_norm_c(const void* y, const void* w_post, const float* res_in, float* res_out, const void* w_next,
@@ -530,4 +569,25 @@ B200_API int b200_sandwich_norm(const void* y, const void* w_post, const float* 
                                 int w_dtype, void* stream) {
   return b200_sandwich_norm_c(y, w_post, res_in, res_out, w_next, h, rows, cols, eps, off, mult, 0, y_dtype, h_dtype, w_dtype,
                               stream);
+}
+
+B200_API int b200_poly_norm(const void* z, const float* act, void* y, long long rows, int cols, float eps, int dtype, void* stream) {
+  using namespace b200;
+  if (rows <= 0) return 0;
+  if (cols <= 0) return B200_ERR_BAD_SHAPE;
+  cudaStream_t st = (cudaStream_t)stream;
+  const int V = dtype == B200_DT_FP32 ? 4 : 8;
+  const bool vec = cols % V == 0 && !((reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(y)) & 15);
+#define PN(T, VV)                                                                                                            \
+  do {                                                                                                                       \
+    if (vec) poly_norm_kernel<T, VV><<<(unsigned)rows, 256, 0, st>>>((const T*)z, act, (T*)y, cols, eps);                     \
+    else poly_norm_kernel<T, 1><<<(unsigned)rows, 256, 0, st>>>((const T*)z, act, (T*)y, cols, eps);                          \
+  } while (0)
+  if (dtype == B200_DT_BF16) PN(__nv_bfloat16, 8);
+  else if (dtype == B200_DT_FP16) PN(__half, 8);
+  else if (dtype == B200_DT_FP32) PN(float, 4);
+  else return B200_ERR_UNSUPPORTED;
+#undef PN
+  B200_LAUNCH_CHECK();
+  return 0;
 }

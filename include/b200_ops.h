@@ -499,14 +499,15 @@ int b200_moe_route_grouped(const void* h, const void* wr, const float* corr, lon
                            long long tokens, int W, int E, int X, int top, int groups, int keep, int group_top, int renorm,
                            int softmax, int h_dtype, int w_dtype, void* stream);
 /* Expert-sorted, tile-padded layout of the assignments top_i int64 [assignments] (= tokens * top): dest int64 [assignments],
- * tok int64 [assignments] (= r / top), tile_map int32 [n_tiles] (expert of a row tile, -1 past the last), counts int64 [E].
+ * tok int64 [assignments] (= r / top; ids of E and above get no row: dest -1), tile_map int32 [n_tiles] (expert of a row tile, -1 past the last), counts int64 [E].
  * B200_ERR_UNSUPPORTED when the ids do not fit in shared memory (about 100k assignments). */
 int b200_moe_dispatch(const long long* top_i, long long* dest, long long* tok, int* tile_map, long long* counts,
                       long long assignments, int E, int top, int tile, int n_tiles, void* stream);
 /* out fp32 [tokens, W] = sum_k p[t, k] * y[dest[t * top + k]] (y: expert-sorted rows of a grouped GEMM), plus
- * gate[t] * shared[t] when shared ([tokens, W], y's dtype) is given (gate fp32 [tokens] or NULL = 1). */
-int b200_moe_combine(const void* y, const long long* dest, const float* p, const void* shared, const float* gate, float* out,
-                     long long tokens, int W, int top, int dtype, void* stream);
+ * gate[t] * shared[t] when shared ([tokens, W], y's dtype) is given (gate fp32 [tokens] or NULL = 1). dest -1: an identity
+ * expert, which adds p * ident[t] (fp32 [tokens, W]; NULL: nothing). */
+int b200_moe_combine(const void* y, const long long* dest, const float* p, const void* shared, const float* gate,
+                     const float* ident, float* out, long long tokens, int W, int top, int dtype, void* stream);
 /* y [rows, F] = act(gate) * up over gu [rows, 2F] (gate | up); act 0: silu, 1: tanh-form GELU, 2: erf GELU. */
 int b200_act_glu(const void* gu, void* y, long long rows, int F, int act, int dtype, void* stream);
 
@@ -563,19 +564,19 @@ int b200_qknorm_rope_store(const float* proj, long long ld, const float* wq, con
                            const float* sin_t, const int* pos, const int* slot, const int* table, int max_blocks, void* q_out,
                            void* ck, void* cv, int tokens, int H, int G, int M, int D, int Dv, int rot, int block_size, float eps,
                            int has_kv, int dtype, void* stream);
-/* out [tokens, H * Dv]: token t sees key j <= pos[t] of its row if pos[t] - j < window or j < keep_first (window <= 0: all).
+/* out, rows of stride ldo holding H * Dv: token t sees key j <= pos[t] of its row if pos[t] - j < window or j < keep_first (window <= 0: all).
  * Each of the M maps is a softmax attention over the same values; combine (M = 2): o = a_0 - lambda a_1, then
- * o / sqrt(mean(o^2) + eps) * post. Dv <= 256. fp32 arithmetic. nsplit > 1 cuts every token's visible keys into ranges
+ * o / sqrt(mean(o^2) + eps); the result is multiplied by post. Dv <= 256. fp32 arithmetic. nsplit > 1 cuts every token's visible keys into ranges
  * (part: fp32 [tokens, H, M, nsplit, Dv + 2] scratch). */
 int b200_multimap_attn(const void* q, const void* ck, const void* cv, const int* pos, const int* slot, const int* table,
-                       int max_blocks, void* out, float* part, int tokens, int H, int G, int M, int D, int Dv, int block_size,
+                       int max_blocks, void* out, long long ldo, float* part, int tokens, int H, int G, int M, int D, int Dv, int block_size,
                        float scale, int window, int keep_first, int nsplit, int combine, float lambda, float post, float eps,
                        int dtype, void* stream);
 /* The same for bf16 prompt pieces on mma.sync: tiles int32 [n_tiles, 4] = (first row, rows <= 64, position of the first row,
  * cache row). D in {32, 48, 64, 96, 128}, Dv in {32, 64, 96, 128}, block_size a power of two, scale > 0; else
  * B200_ERR_UNSUPPORTED (use b200_multimap_attn). */
 int b200_multimap_attn_mma(const void* q, const void* ck, const void* cv, const int* tiles, int n_tiles, const int* table,
-                           int max_blocks, void* out, int H, int G, int M, int D, int Dv, int block_size, float scale, int window,
+                           int max_blocks, void* out, long long ldo, int H, int G, int M, int D, int Dv, int block_size, float scale, int window,
                            int keep_first, int combine, float lambda, float post, float eps, int dtype, void* stream);
 
 /* ---- talking-heads attention over the paged key cache (csrc/talking_attn.cu): raw_g = scale q_g . k - r1[g] log(1 + r2[g]
@@ -600,13 +601,14 @@ int b200_talking_attn_mma(const void* q, long long ldq, const void* gate, long l
  * state row) or NULL (every token its own run, from pos / slot). A run at position 0 starts from zero state. ---- */
 int b200_short_conv(const float* x, long long ldx, const float* w, const float* state, const int* pos, const int* slot, float* y,
                     long long ldy, int tokens, int C, int taps, int act, void* stream);
-/* The same with a bias per channel (or NULL), `residual` 1: y = x + act(conv(x) + bias), and y in y_dtype (fp32 / bf16). */
-int b200_short_conv_ex(const float* x, long long ldx, const float* w, const float* bias, const float* state, const int* pos,
-                       const int* slot, void* y, long long ldy, int tokens, int C, int taps, int act, int residual, int y_dtype,
-                       void* stream);
+/* The same with a bias per channel (or NULL), `residual` 1: y = x + act(conv(x) + bias), x in x_dtype and y in y_dtype
+ * (fp32 / bf16). step_tail 1: every token is a run of its own and its tail is advanced in the same launch. */
+int b200_short_conv_ex(const void* x, long long ldx, const float* w, const float* bias, float* state, const int* pos,
+                       const int* slot, void* y, long long ldy, int tokens, int C, int taps, int act, int residual, int step_tail,
+                       int x_dtype, int y_dtype, void* stream);
 int b200_silu_rows(float* x, long long ld, long long rows, int cols, void* stream);
-int b200_short_conv_tail(const float* x, long long ldx, float* state, const int* runs, const int* pos, const int* slot, int n_runs,
-                         int C, int taps, void* stream);
+int b200_short_conv_tail(const void* x, long long ldx, const float* in_bias, float* state, const int* runs, const int* pos,
+                         const int* slot, int n_runs, int C, int taps, int x_dtype, void* stream);
 int b200_delta_gates(float* q, long long ldq, float* k, long long ldk, float* a, long long lda, float* b, long long ldb,
                      const float* dt_bias, const float* A_log, int tokens, int G, int H, int D, float qscale, float unit_eps,
                      void* stream);
@@ -628,10 +630,44 @@ int b200_ssm_gates(const float* dt, long long ld, const float* dt_bias, const fl
                    int H, void* stream);
 /* Per token: v = o[h, d] * oscale; e != NULL: v /= max(|o[h, Dv] * oscale|, e[t, h]) + den_eps; skip != NULL: v += skip[h] x[c];
  * pre != NULL: v *= silu(pre[c]); RMS norm over `groups` equal column groups; times w (w_full 1: [H * Dv], 0: [group size]);
- * post != NULL: v *= sigmoid(post[c]). o fp32 [tokens, H, ocols]; out [tokens, H * Dv] in out_dtype. */
+ * post != NULL: v *= sigmoid(post[c]), or silu(post[c]) with post_silu 1. o fp32 [tokens, H, ocols]; out [tokens, H * Dv] in out_dtype. */
 int b200_scan_readout(const float* o, int ocols, const float* e, float den_eps, float oscale, const float* skip, const float* x,
-                      long long ldx, const float* pre, long long ldpre, const float* post, long long ldpost, const float* w,
-                      int w_full, void* out, long long tokens, int H, int Dv, int groups, float eps, int out_dtype, void* stream);
+                      long long ldx, const float* pre, long long ldpre, const float* post, long long ldpost, int post_silu,
+                      const float* w, int w_full, void* out, long long tokens, int H, int Dv, int groups, float eps, int out_dtype, void* stream);
+
+/* Per-channel decays of a low-rank input and the scan that uses them (csrc/channel_scan.cu): out[t, c] = sigmoid(w2[c] . x[t] +
+ * bias[c])^inv_tau; per head S <- diag(g) S + k v^T, o = S^T q (fp32). n_tiles > 0: runs are walked tile by tile in parallel,
+ * tiles int32 [n_tiles, 4] = (first row, rows, first position, state row), tile_of [n_tiles, 4] = (run, place in the run, tiles
+ * of the run, its first tile), run_tiles [n_runs, 4] = (first tile, tiles, 0, 0), part fp32 [n_tiles, H, D, Dv] and pdec fp32
+ * [n_tiles, H, D] are scratch. chunk: tokens staged at a time (at most 16). */
+int b200_lowrank_decay(const float* x, long long ldx, const float* w2, const float* bias, float* out, int tokens, int C, int rank,
+                       float inv_tau, void* stream);
+int b200_channel_scan(const float* q, long long ldq, const float* k, long long ldk, const float* v, long long ldv, const float* g,
+                      long long ldg, float* state, float* part, float* pdec, const int* runs, int n_runs, const int* tiles,
+                      int n_tiles, const int* tile_of, const int* run_tiles, int chunk, const int* pos, const int* slot, float* o,
+                      int H, int G, int D, int Dv, void* stream);
+/* Selective state space with a decay per channel and state (csrc/selective_scan.cu): s = softplus(dt + dt_bias), S[n, c] <-
+ * exp(s_c A[n, c]) S[n, c] + s_c u_c B_n, y_c = (sum_n S[n, c] C_n + D_c u_c) silu(gate_c) scale. u, B, C, gate and y in `dtype`,
+ * the rest fp32; state [rows, N, inner]; A [N, inner]; tiles as above, part fp32 [n_tiles * (N + 1) * inner]. */
+int b200_selective_scan(const void* u, long long ldu, const float* dt, long long lddt, const float* dt_bias, const void* B,
+                        long long ldB, const void* C, long long ldC, const float* A, const float* D, float* state, float* part,
+                        const void* gate, long long ldg, float scale, void* y, long long ldy, const int* runs, int n_runs,
+                        const int* tiles, int n_tiles, const int* tile_of, const int* run_tiles, const int* pos, const int* slot,
+                        int inner, int N, int dtype, void* stream);
+
+/* y = act[0] N(z) + act[1] N(z^2) + act[2] N(z^3) + act[3] per row, N(v) = v / sqrt(mean(v^2) + eps) (csrc/norm.cu). */
+int b200_poly_norm(const void* z, const float* act, void* y, long long rows, int cols, float eps, int dtype, void* stream);
+
+/* q | k | v rows of one-map attention (csrc/multimap_attn.cu): bias, a causal convolution per channel (w [C, taps]; tail fp32
+ * [rows, taps - 1, C] holds the biased inputs before a run), row-wise RMS norms without a weight, q times
+ * 1 + temp_coef ln(floor((p + 1) / temp_every) + 1); q to q_out, k and v to their pages. taps <= 5, D and Dv <= 512. */
+int b200_conv_qknorm_store(const void* proj, long long ld, const float* bias, const float* w, const float* tail, const int* pos,
+                           const int* slot, const int* table, int max_blocks, void* q_out, void* ck, void* cv, int tokens, int H,
+                           int G, int D, int Dv, int taps, int block_size, float eps, float temp_coef, float temp_every, int norm_qk,
+                           int norm_v, int x_dtype, int dtype, void* stream);
+/* xs[dest[r]] = h[tok[r]] for the assignments r with a row (dest >= 0) */
+int b200_moe_gather(const void* h, const long long* dest, const long long* tok, void* xs, long long assignments, long long row_bytes,
+                    void* stream);
 
 #ifdef __cplusplus
 }

@@ -35,6 +35,9 @@ class Pieces:
     longest: int                    # tokens of the longest run
     runs: Optional[torch.Tensor] = None     # int32 [n_runs, 4] = (first row, rows, position of the first row, cache row): whole runs,
     n_runs: int = 0                         # walked in order by the recurrent mixers (ops.linear_scan)
+    tile_of: Optional[torch.Tensor] = None  # int32 [n_tiles, 4] = (run, place in the run, tiles of the run, the run's first tile)
+    run_tiles: Optional[torch.Tensor] = None    # int32 [n_runs, 4] = (first tile, tiles, 0, 0)
+    tile_rows: int = TILE_Q                 # tokens of every tile of a run but its last
 
     def use_mma(self, q: torch.Tensor, head_dim: int, window: int, scale: float = 1.0) -> bool:
         return (self.longest >= 8 and scale > 0 and q.dtype == torch.bfloat16 and head_dim % 16 == 0 and head_dim <= 128
@@ -46,9 +49,16 @@ def make_pieces(runs: Sequence[Sequence[int]], device) -> Pieces:
     the recurrent mixers) and cut into tiles of at most ``TILE_Q`` rows (for the tensor-core attention kernels)."""
     runs = [[int(v) for v in r] for r in runs if r[1] > 0]
     tiles = [[first + q0, min(TILE_Q, n - q0), p0 + q0, row] for first, n, p0, row in runs for q0 in range(0, n, TILE_Q)]
-    tl = torch.tensor(tiles + runs, dtype=torch.int32)
+    tile_of: List[List[int]] = []
+    run_tiles: List[List[int]] = []
+    for r, run in enumerate(runs):
+        nt, at = -(-run[1] // TILE_Q), len(tile_of)
+        tile_of += [[r, j, nt, at] for j in range(nt)]
+        run_tiles.append([at, nt, 0, 0])
+    tl = torch.tensor(tiles + runs + tile_of + run_tiles, dtype=torch.int32)
     tl = tl.pin_memory().to(device, non_blocking=True) if torch.device(device).type == "cuda" else tl
-    return Pieces(tl[:len(tiles)], len(tiles), max((r[1] for r in runs), default=0), tl[len(tiles):], len(runs))
+    nt, nr = len(tiles), len(runs)
+    return Pieces(tl[:nt], nt, max((r[1] for r in runs), default=0), tl[nt:nt + nr], nr, tl[nt + nr:2 * nt + nr], tl[2 * nt + nr:])
 
 
 Entry = Tuple[int, int, Sequence[int], Sequence[int]]       # (cache row, first position, tokens, wanted indices into tokens)
@@ -98,6 +108,12 @@ class RaggedGenerator(Generator):
                 n += k
         return n
 
+    def _check_position(self, p: int) -> None:
+        """Models with a position table have a last position; the table is read on the device, so it is guarded here."""
+        limit = getattr(self.model, "max_positions", 0)
+        if limit and p >= limit:
+            raise ValueError(f"position {p} is past the model's last position {limit - 1}")
+
     # ------------------------------------------------------------------ the step
     @torch.no_grad()
     def step(self, entries: Sequence[Entry], cache: PagedKVCache, layer_outputs: Optional[list] = None) -> Optional[torch.Tensor]:
@@ -120,6 +136,7 @@ class RaggedGenerator(Generator):
                 continue
             if pos0 + n > cache.max_len:
                 raise ValueError(f"sequence of {pos0 + n} tokens does not fit the cache rows of {cache.max_len}")
+            self._check_position(pos0 + n - 1)
             base = len(ids)
             ids.extend(int(t) for t in toks)
             pos.extend(range(pos0, pos0 + n))
@@ -149,6 +166,7 @@ class RaggedGenerator(Generator):
         the bucket write to the cache's scratch row. Returns fp32 logits [len(tokens), vocab]."""
         dev = self.model.embed_tokens.device
         n = len(tokens)
+        self._check_position(max(positions))
         nb = 1
         while nb < n:
             nb *= 2

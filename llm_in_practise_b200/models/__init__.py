@@ -26,6 +26,11 @@ def _load_kudonex(path, dtype, device):
     return kudonex_from_pretrained(path, dtype=dtype, device=device)
 
 
+def _load_lorenex(path, dtype, device):
+    from .lorenex import lorenex_from_pretrained
+    return lorenex_from_pretrained(path, dtype=dtype, device=device)
+
+
 # ``architecture`` (or HF ``model_type`` / ``architectures[0]``) of config.json -> loader(path, dtype, device).
 # Anything not listed is read as a Qwen2/Qwen3-style HF checkpoint by ``io.hf.from_pretrained``.
 MODEL_REGISTRY: Dict[str, Callable] = {
@@ -37,6 +42,8 @@ MODEL_REGISTRY: Dict[str, Callable] = {
     "duratar": _load_duratar,
     "Kudonex": _load_kudonex,
     "kudonex": _load_kudonex,
+    "Lorenex": _load_lorenex,
+    "lorenex": _load_lorenex,
 }
 
 

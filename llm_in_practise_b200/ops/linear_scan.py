@@ -13,6 +13,9 @@ run that starts at position 0 starts from a zero state, so state rows are reused
     linear_scan    mode "decay":  S <- decay_h S + k v^T;                                  o = S^T q
                    mode "delta":  S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T;    o = S^T q
                    mode "gated":  S <- a_t S + b_t k v^T (one a, b per token and head);    o = S^T q
+                   mode "channel": S <- diag(g) S + k v^T (a decay per key channel);       o = S^T q
+    lowrank_decay  per-channel decays sigmoid(W_2 x + bias)^(1 / tau) of a low-rank input x
+    selective_scan S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c u_c B_n; y_c = sum_n S[c, n] C_n + D_c u_c; y silu(gate) scale
     mlstm_gates    capped log gates of an mLSTM and their running maximum -> (a, b, exp(-m)) for the gated scan
     ssm_gates      dt = softplus(x + bias), a = exp(-exp(A_log) dt), b = dt: the step sizes of a selective state space
     scan_readout   normaliser division / skip term / silu gate, RMS norm over column groups, weight, sigmoid gate
@@ -41,22 +44,24 @@ def _run_list(runs, pos, slot):
 def short_conv(x: torch.Tensor, w: torch.Tensor, tail: torch.Tensor, pos: torch.Tensor, slot: torch.Tensor,
                runs: Optional[torch.Tensor], n_runs: int, act: bool = True, bias: Optional[torch.Tensor] = None,
                residual: bool = False, out_dtype: torch.dtype = torch.float32) -> torch.Tensor:
-    """``x`` fp32 [T, C] (rows may be strided) -> y [T, C] in ``out_dtype`` (fp32 / bf16); ``w`` fp32 [C, taps] (last column
-    weighs the current token), ``bias`` fp32 [C] or None; ``tail`` fp32 [rows, taps - 1, C] is read for the inputs before each
-    run and then advanced over the run. ``residual``: y = x + act(conv(x) + bias)."""
+    """``x`` fp32 or bf16 [T, C] (rows may be strided) -> y [T, C] in ``out_dtype`` (fp32 / bf16); ``w`` fp32 [C, taps] (last
+    column weighs the current token), ``bias`` fp32 [C] or None; ``tail`` fp32 [rows, taps - 1, C] is read for the inputs
+    before each run and then advanced over the run (one launch for a decode batch, two otherwise). ``residual``:
+    y = x + act(conv(x) + bias)."""
     T, C = x.shape
     taps = w.shape[1]
     y = torch.empty(T, C, dtype=out_dtype, device=x.device)
     if nv.use_native(x):
-        if x.dtype != torch.float32 or x.stride(1) != 1:
-            raise ValueError("short_conv: fp32 rows with a contiguous last dim")
-        fn = nv.proto("b200_short_conv_ex", [vp, i64, vp, vp, vp, vp, vp, vp, i64, i32, i32, i32, i32, i32, i32, vp])
+        if x.dtype not in (torch.float32, torch.bfloat16) or x.stride(1) != 1:
+            raise ValueError("short_conv: fp32 or bf16 rows with a contiguous last dim")
+        fn = nv.proto("b200_short_conv_ex", [vp, i64, vp, vp, vp, vp, vp, vp, i64, i32, i32, i32, i32, i32, i32, i32, i32, vp])
+        step_tail = runs is None and taps > 1                 # every token is its own run: the thread that read a tail advances it
         nv.check(fn(nv.ptr(x), x.stride(0), nv.ptr(w), nv.ptr(bias), nv.ptr(tail), nv.ptr(pos), nv.ptr(slot), nv.ptr(y), y.stride(0),
-                    T, C, taps, int(act), int(residual), nv.dtype_code(out_dtype), nv.stream()), "short_conv")
-        fn = nv.proto("b200_short_conv_tail", [vp, i64, vp, vp, vp, vp, i32, i32, i32, vp])
-        nv.check(fn(nv.ptr(x), x.stride(0), nv.ptr(tail), nv.ptr(runs), nv.ptr(pos), nv.ptr(slot), n_runs if runs is not None else T,
-                    C, taps, nv.stream()), "short_conv_tail")
-        nv.count_launch(2)
+                    T, C, taps, int(act), int(residual), int(step_tail), nv.dtype_code(x.dtype), nv.dtype_code(out_dtype),
+                    nv.stream()), "short_conv")
+        nv.count_launch()
+        if runs is not None and taps > 1:
+            _conv_tail(x, None, tail, runs, pos, slot, n_runs, C, taps)
         return y
     L = taps - 1
     for first, n, p0, s in _run_list(runs, pos, slot):
@@ -72,6 +77,14 @@ def short_conv(x: torch.Tensor, w: torch.Tensor, tail: torch.Tensor, pos: torch.
         if L:
             tail[s] = ext[n:n + L]
     return y
+
+
+def _conv_tail(x, in_bias, tail, runs, pos, slot, n_runs, C, taps):
+    """Advance ``tail`` over the step's runs (after everything that reads the old tail has been launched)."""
+    fn = nv.proto("b200_short_conv_tail", [vp, i64, vp, vp, vp, vp, vp, i32, i32, i32, i32, vp])
+    nv.check(fn(nv.ptr(x), x.stride(0), nv.ptr(in_bias), nv.ptr(tail), nv.ptr(runs), nv.ptr(pos), nv.ptr(slot), n_runs, C, taps,
+                nv.dtype_code(x.dtype), nv.stream()), "short_conv_tail")
+    nv.count_launch()
 
 
 def silu_rows_(x: torch.Tensor) -> torch.Tensor:
@@ -105,29 +118,50 @@ def delta_gates(q: torch.Tensor, k: torch.Tensor, a: torch.Tensor, b: torch.Tens
     b.copy_(torch.sigmoid(b))
 
 
+SCAN_MODES = ("decay", "delta", "gated", "channel")
+
+
 def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, pos: torch.Tensor, slot: torch.Tensor,
                 runs: Optional[torch.Tensor], n_runs: int, H: int, G: int, D: int, Dv: int, mode: str,
                 decay: Optional[torch.Tensor] = None, g: Optional[torch.Tensor] = None, beta: Optional[torch.Tensor] = None,
-                act: bool = False, ones: bool = False) -> torch.Tensor:
+                act: bool = False, ones: bool = False, pieces=None) -> torch.Tensor:
     """o fp32 [T, H * Dv]. q, k fp32 [T, G * D] (head h reads head h // (H / G)), v fp32 [T, H * Dv] (rows may be strided);
     ``state`` fp32 [rows, H, D, Dv] is read at the start of each run and written at its end. ``mode`` "decay" takes
     ``decay`` fp32 [H]; "delta" takes ``g`` fp32 [T, H * D] (per key channel) and ``beta`` fp32 [T, H]; "gated" takes
-    ``g`` = a and ``beta`` = b, both fp32 [T, H]. ``act``: silu on q, k and v as they are read. ``ones``: every head of v gets
+    ``g`` = a and ``beta`` = b, both fp32 [T, H]; "channel" takes ``g`` fp32 [T, H * D] alone. ``act``: silu on q, k and v as they are read. ``ones``: every head of v gets
     one more column, all ones — ``Dv`` counts it, v itself has ``Dv - 1`` columns per head — so the state's last column
-    accumulates the decayed b k alone and o's last column is its product with q."""
+    accumulates the decayed b k alone and o's last column is its product with q. ``pieces`` (``inference.ragged.Pieces``,
+    mode "channel"): runs of several tiles are walked tile by tile in parallel, see ``csrc/linear_scan.cu``."""
     T = q.shape[0]
     o = torch.empty(T, H * Dv, dtype=torch.float32, device=q.device)
     delta = mode == "delta"
     gated = mode == "gated"
-    if mode not in ("decay", "delta", "gated"):
+    channel = mode == "channel"
+    if mode not in SCAN_MODES:
         raise ValueError(f"linear_scan: no mode {mode!r}")
+    if nv.use_native(q) and channel:
+        if act or ones:
+            raise ValueError("linear_scan: mode \"channel\" takes neither act nor ones")
+        tiled = pieces is not None and pieces.tile_of is not None and pieces.longest > pieces.tile_rows
+        nt = pieces.n_tiles if tiled else 0
+        part = torch.empty(nt * H * D * Dv, dtype=torch.float32, device=q.device) if tiled else None
+        pdec = torch.empty(nt * H * D, dtype=torch.float32, device=q.device) if tiled else None
+        longest = 1 if runs is None else (pieces.longest if pieces is not None else 16)
+        opt = lambda name: nv.ptr(getattr(pieces, name) if tiled else None)                      # noqa: E731
+        fn = nv.proto("b200_channel_scan", [vp, i64, vp, i64, vp, i64, vp, i64, vp, vp, vp, vp, i32, vp, i32, vp, vp, i32, vp, vp, vp,
+                                            i32, i32, i32, i32, vp])
+        nv.check(fn(nv.ptr(q), q.stride(0), nv.ptr(k), k.stride(0), nv.ptr(v), v.stride(0), nv.ptr(g), g.stride(0), nv.ptr(state),
+                    nv.ptr(part), nv.ptr(pdec), nv.ptr(runs), n_runs if runs is not None else T, opt("tiles"), nt, opt("tile_of"),
+                    opt("run_tiles"), longest, nv.ptr(pos), nv.ptr(slot), nv.ptr(o), H, G, D, Dv, nv.stream()), "channel_scan")
+        nv.count_launch(3 if tiled else 1)
+        return o
     if nv.use_native(q):
         fn = nv.proto("b200_linear_scan", [vp, i64, vp, i64, vp, i64, vp, i64, vp, i64, vp, vp, vp, vp, vp, i32, vp, i32, i32, i32,
                                            i32, i32, i32, i32, vp])
         per = delta or gated
         nv.check(fn(nv.ptr(q), q.stride(0), nv.ptr(k), k.stride(0), nv.ptr(v), v.stride(0), nv.ptr(g), g.stride(0) if per else 0,
-                    nv.ptr(beta), beta.stride(0) if per else 0, nv.ptr(decay), nv.ptr(state), nv.ptr(runs), nv.ptr(pos),
-                    nv.ptr(slot), n_runs if runs is not None else T, nv.ptr(o), H, G, D, Dv, 2 if gated else int(delta), int(act),
+                    nv.ptr(beta), beta.stride(0) if beta is not None else 0, nv.ptr(decay), nv.ptr(state), nv.ptr(runs), nv.ptr(pos),
+                    nv.ptr(slot), n_runs if runs is not None else T, nv.ptr(o), H, G, D, Dv, SCAN_MODES.index(mode), int(act),
                     int(ones), nv.stream()), "linear_scan")
         nv.count_launch()
         return o
@@ -148,6 +182,8 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.
                 S = S + kf[t][:, :, None] * u[:, None, :]
             elif gated:
                 S = g[t].float().view(H, 1, 1) * S + kf[t][:, :, None] * (beta[t].float().view(H, 1) * vf[t])[:, None, :]
+            elif channel:
+                S = S * g[t].float().reshape(H, D, 1) + kf[t][:, :, None] * vf[t][:, None, :]
             else:
                 S = decay.float().view(H, 1, 1) * S + kf[t][:, :, None] * vf[t][:, None, :]
             ov[t] = torch.einsum("hde,hd->he", S, qf[t])
@@ -202,11 +238,11 @@ def ssm_gates(dt: torch.Tensor, dt_bias: torch.Tensor, A_log: torch.Tensor):
 def scan_readout(o: torch.Tensor, H: int, Dv: int, w: torch.Tensor, groups: int, eps: float, out_dtype: torch.dtype,
                  e: Optional[torch.Tensor] = None, den_eps: float = 0.0, oscale: float = 1.0,
                  skip: Optional[torch.Tensor] = None, x: Optional[torch.Tensor] = None, pre: Optional[torch.Tensor] = None,
-                 post: Optional[torch.Tensor] = None) -> torch.Tensor:
+                 post: Optional[torch.Tensor] = None, post_act: str = "sigmoid") -> torch.Tensor:
     """What follows a scan, per token, in one pass: ``o`` fp32 [T, H * ocols] with ocols = Dv, or Dv + 1 when the scan carried
     a column of ones (``e`` fp32 [T, H] given: v = oscale o[h, :Dv] / (max(|oscale o[h, Dv]|, e[h]) + den_eps)); ``skip`` fp32
     [H] with ``x`` fp32 [T, H * Dv]: v += skip[h] x; ``pre``: v *= silu(pre); RMS norm over ``groups`` equal parts of the
-    H * Dv columns; times ``w`` (fp32, one per column, or one per column of a group); ``post``: v *= sigmoid(post). pre / post /
+    H * Dv columns; times ``w`` (fp32, one per column, or one per column of a group); ``post``: v *= sigmoid(post), or silu(post) with ``post_act`` "silu". pre / post /
     x are fp32 rows that may be strided. Returns [T, H * Dv] in ``out_dtype``."""
     T = o.shape[0]
     N = H * Dv
@@ -214,11 +250,11 @@ def scan_readout(o: torch.Tensor, H: int, Dv: int, w: torch.Tensor, groups: int,
     w_full = w.numel() == N
     if nv.use_native(o):
         out = torch.empty(T, N, dtype=out_dtype, device=o.device)
-        fn = nv.proto("b200_scan_readout", [vp, i32, vp, f32, f32, vp, vp, i64, vp, i64, vp, i64, vp, i32, vp, i64, i32, i32, i32,
+        fn = nv.proto("b200_scan_readout", [vp, i32, vp, f32, f32, vp, vp, i64, vp, i64, vp, i64, i32, vp, i32, vp, i64, i32, i32, i32,
                                             f32, i32, vp])
         st = lambda z: z.stride(0) if z is not None else 0                      # noqa: E731
         nv.check(fn(nv.ptr(o), ocols, nv.ptr(e), float(den_eps), float(oscale), nv.ptr(skip), nv.ptr(x), st(x), nv.ptr(pre), st(pre),
-                    nv.ptr(post), st(post), nv.ptr(w), int(w_full), nv.ptr(out), T, H, Dv, groups, float(eps),
+                    nv.ptr(post), st(post), int(post_act == "silu"), nv.ptr(w), int(w_full), nv.ptr(out), T, H, Dv, groups, float(eps),
                     nv.dtype_code(out_dtype), nv.stream()), "scan_readout")
         nv.count_launch()
         return out
@@ -235,5 +271,72 @@ def scan_readout(o: torch.Tensor, H: int, Dv: int, w: torch.Tensor, groups: int,
     v = (v * torch.rsqrt((v * v).mean(-1, keepdim=True) + eps)).reshape(T, N)
     v = v * (w.float() if w_full else w.float().repeat(groups))
     if post is not None:
-        v = v * torch.sigmoid(post.float())
+        v = v * (F.silu(post.float()) if post_act == "silu" else torch.sigmoid(post.float()))
     return v.to(out_dtype)
+
+
+def lowrank_decay(x: torch.Tensor, w2: torch.Tensor, bias: torch.Tensor, tau: float) -> torch.Tensor:
+    """``x`` fp32 [T, r] (rows may be strided), ``w2`` fp32 [C, r], ``bias`` fp32 [C] -> sigmoid(w2 x + bias)^(1 / tau), fp32
+    [T, C], formed as exp(log sigmoid(.) / tau)."""
+    T, r = x.shape
+    C = w2.shape[0]
+    if nv.use_native(x):
+        if x.dtype != torch.float32 or x.stride(1) != 1:
+            raise ValueError("lowrank_decay: fp32 rows with a contiguous last dim")
+        out = torch.empty(T, C, dtype=torch.float32, device=x.device)
+        fn = nv.proto("b200_lowrank_decay", [vp, i64, vp, vp, vp, i32, i32, i32, f32, vp])
+        nv.check(fn(nv.ptr(x), x.stride(0), nv.ptr(w2), nv.ptr(bias), nv.ptr(out), T, C, r, 1.0 / float(tau), nv.stream()), "lowrank_decay")
+        nv.count_launch()
+        return out
+    z = x.float() @ w2.float().t() + bias.float()
+    return torch.exp(F.logsigmoid(z) / tau)
+
+
+def selective_scan(u: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, Bm: torch.Tensor, Cm: torch.Tensor, A: torch.Tensor,
+                   D: torch.Tensor, state: torch.Tensor, pos: torch.Tensor, slot: torch.Tensor, runs: Optional[torch.Tensor],
+                   n_runs: int, gate: Optional[torch.Tensor] = None, scale: float = 1.0, out: Optional[torch.Tensor] = None,
+                   pieces=None) -> torch.Tensor:
+    """A selective state space with a decay per channel and state. ``u`` [T, I], ``Bm`` / ``Cm`` [T, N] and ``gate`` [T, I] in one
+    dtype (fp32 / bf16, rows may be strided), ``dt`` fp32 [T, I] before ``dt_bias`` fp32 [I] and softplus, ``A`` fp32 [N, I]
+    (negative rates), ``D`` fp32 [I], ``state`` fp32 [rows, N, I] read at the start of each run and written at its end:
+
+        s = softplus(dt + dt_bias);  S[n, c] <- exp(s_c A[n, c]) S[n, c] + s_c u_c B_n
+        y_c = (sum_n S[n, c] C_n + D_c u_c) silu(gate_c) scale
+
+    Returns y [T, I] in u's dtype (``out``: where to write it, rows may be strided). ``pieces``: runs of several tiles are
+    walked tile by tile in parallel (local states, a carry over the tiles of a run, then the outputs)."""
+    T, inner = u.shape
+    N = A.shape[0]
+    y = out if out is not None else torch.empty(T, inner, dtype=u.dtype, device=u.device)
+    if nv.use_native(u):
+        for t in (u, Bm, Cm, y) + ((gate,) if gate is not None else ()):
+            if t.dtype != u.dtype or t.stride(1) != 1:
+                raise ValueError("selective_scan: u, B, C, gate and out share a dtype and have contiguous last dims")
+        if dt.dtype != torch.float32 or dt.stride(1) != 1:
+            raise ValueError("selective_scan: dt fp32 rows with a contiguous last dim")
+        tiled = pieces is not None and pieces.tile_of is not None and pieces.longest > pieces.tile_rows
+        part = torch.empty(pieces.n_tiles * (N + 1) * inner, dtype=torch.float32, device=u.device) if tiled else None
+        fn = nv.proto("b200_selective_scan", [vp, i64, vp, i64, vp, vp, i64, vp, i64, vp, vp, vp, vp, vp, i64, f32, vp, i64, vp, i32, vp,
+                                              i32, vp, vp, vp, vp, i32, i32, i32, vp])
+        nv.check(fn(nv.ptr(u), u.stride(0), nv.ptr(dt), dt.stride(0), nv.ptr(dt_bias), nv.ptr(Bm), Bm.stride(0), nv.ptr(Cm), Cm.stride(0),
+                    nv.ptr(A), nv.ptr(D), nv.ptr(state), nv.ptr(part), nv.ptr(gate), gate.stride(0) if gate is not None else 0, float(scale),
+                    nv.ptr(y), y.stride(0), nv.ptr(runs), n_runs if runs is not None else T,
+                    nv.ptr(pieces.tiles if tiled else None), pieces.n_tiles if tiled else 0, nv.ptr(pieces.tile_of if tiled else None),
+                    nv.ptr(pieces.run_tiles if tiled else None), nv.ptr(pos), nv.ptr(slot), inner, N, nv.dtype_code(u.dtype), nv.stream()), "selective_scan")
+        nv.count_launch(3 if tiled else 1)
+        return y
+    z = dt.float() + dt_bias.float()
+    s = z.clamp(min=0) + torch.log1p(torch.exp(-z.abs()))
+    uf, Bf, Cf = u.float(), Bm.float(), Cm.float()
+    acc = torch.empty(T, inner, dtype=torch.float32, device=u.device)
+    for first, n, p0, r in _run_list(runs, pos, slot):
+        S = state[r].clone() if p0 > 0 else torch.zeros(N, inner, dtype=torch.float32, device=u.device)
+        for t in range(first, first + n):
+            S = torch.exp(s[t][None, :] * A) * S + (s[t] * uf[t])[None, :] * Bf[t][:, None]
+            acc[t] = (S * Cf[t][:, None]).sum(0)
+        state[r] = S
+    acc = acc + D.float() * uf
+    if gate is not None:
+        acc = acc * F.silu(gate.float())
+    y.copy_((acc * scale).to(u.dtype))
+    return y

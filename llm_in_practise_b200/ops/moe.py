@@ -47,7 +47,8 @@ class Dispatch:
 
 
 def dispatch(top_i: torch.Tensor, num_experts: int, tile: int = TILE) -> Dispatch:
-    """top_i [T, k] expert indices -> expert-sorted, tile-padded row layout. Device ops only."""
+    """top_i [T, k] expert indices -> expert-sorted, tile-padded row layout. Device ops only. Indices of ``num_experts`` and
+    above belong to no expert with weights (identity experts): they get no row (``dest`` -1) and are counted nowhere."""
     T, k = top_i.shape
     R, E = T * k, num_experts
     dev = top_i.device
@@ -72,10 +73,11 @@ def dispatch(top_i: torch.Tensor, num_experts: int, tile: int = TILE) -> Dispatc
     seg_start = seg_end - padc
     start_unp = torch.cumsum(counts, 0) - counts
     order = torch.argsort(flat_e, stable=True)
-    sorted_e = flat_e.index_select(0, order)
+    sorted_e = flat_e.index_select(0, order).clamp_max(E - 1)       # indices past the last expert sort behind all others
     rank_in = torch.arange(R, device=dev) - start_unp.index_select(0, sorted_e)
     dest = torch.empty(R, dtype=torch.long, device=dev)
     dest.index_copy_(0, order, seg_start.index_select(0, sorted_e) + rank_in)
+    dest = torch.where(flat_e < E, dest, torch.full_like(dest, -1))
     tile_start = torch.arange(nt, device=dev) * tile
     e_of_tile = torch.searchsorted(seg_end, tile_start, right=True)
     tile_map = torch.where(tile_start < seg_end[-1], e_of_tile, torch.full_like(e_of_tile, -1)).to(torch.int32)
@@ -262,10 +264,11 @@ route_sigmoid_grouped = route_grouped          # the name its first user (a sigm
 
 
 def moe_combine(y: torch.Tensor, dest: torch.Tensor, top_p: torch.Tensor, shared: Optional[torch.Tensor] = None,
-                gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                gate: Optional[torch.Tensor] = None, identity: Optional[torch.Tensor] = None) -> torch.Tensor:
     """fp32 [T, D]: ``sum_k top_p[t, k] * y[dest[t * top + k]]`` over the expert-sorted rows ``y`` of a grouped GEMM, plus
     ``gate[t] * shared[t]`` when a shared expert's output ``shared`` [T, D] (y's dtype) is given (``gate`` fp32 [T] or [T, 1];
-    None = 1)."""
+    None = 1). An assignment without a row (``dest`` -1: an identity expert) adds ``top_p * identity[t]`` instead (``identity``
+    fp32 [T, D])."""
     T, top = top_p.shape
     W = y.shape[1]
     if nv.use_native(y):
@@ -275,27 +278,49 @@ def moe_combine(y: torch.Tensor, dest: torch.Tensor, top_p: torch.Tensor, shared
             if shared.dtype != y.dtype:
                 raise TypeError("the shared expert's rows must have the routed rows' dtype")
         vp, i32, i64 = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong
-        fn = nv.proto("b200_moe_combine", [vp, vp, vp, vp, vp, vp, i64, i32, i32, i32, vp])
-        nv.check(fn(nv.ptr(y), nv.ptr(dest), nv.ptr(top_p), nv.ptr(shared), nv.ptr(gate), nv.ptr(out), T, W, top, nv.dtype_code(y.dtype),
+        if identity is not None and (identity.dtype != torch.float32 or not identity.is_contiguous()):
+            raise TypeError("moe_combine: the identity experts' rows are contiguous fp32")
+        fn = nv.proto("b200_moe_combine", [vp, vp, vp, vp, vp, vp, vp, i64, i32, i32, i32, vp])
+        nv.check(fn(nv.ptr(y), nv.ptr(dest), nv.ptr(top_p), nv.ptr(shared), nv.ptr(gate), nv.ptr(identity), nv.ptr(out), T, W, top, nv.dtype_code(y.dtype),
                     nv.stream()), "moe_combine")
         nv.count_launch()
         return out
-    out = (y.index_select(0, dest).float().view(T, top, W) * top_p.unsqueeze(-1)).sum(1)
+    rows = y.index_select(0, dest.clamp_min(0)).float().view(T, top, W)
+    if identity is not None:
+        rows = torch.where((dest < 0).view(T, top, 1), identity.float().view(T, 1, W), rows)
+    out = (rows * top_p.unsqueeze(-1)).sum(1)
     if shared is not None:
         out = out + (shared.float() * gate.float().view(T, 1) if gate is not None else shared.float())
     return out
 
 
+def gather_rows(h: torch.Tensor, d: Dispatch) -> torch.Tensor:
+    """The expert-sorted, tile-padded operand of the grouped GEMMs: row ``dest[r]`` is ``h[tok[r]]``. The padding rows of a
+    segment are never read back; the CUDA path leaves them as they are, the other one zero."""
+    if nv.use_native(h) and nv.has("b200_moe_gather"):
+        h = h.contiguous()
+        xs = torch.empty(d.rows, h.shape[1], dtype=h.dtype, device=h.device)
+        vp, i32, i64 = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong
+        fn = nv.proto("b200_moe_gather", [vp, vp, vp, vp, i64, i64, vp])
+        nv.check(fn(nv.ptr(h), nv.ptr(d.dest), nv.ptr(d.tok), nv.ptr(xs), d.dest.numel(), h.shape[1] * h.element_size(), nv.stream()),
+                 "moe_gather")
+        nv.count_launch()
+        return xs
+    xs = torch.zeros(d.rows + 1, h.shape[1], dtype=h.dtype, device=h.device)      # the last row takes what no expert takes
+    return xs.index_copy(0, torch.where(d.dest < 0, d.rows, d.dest), h.index_select(0, d.tok))[:d.rows]
+
+
 def gated_moe_ffn(h: torch.Tensor, top_i: torch.Tensor, top_p: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor,
-                  act, tile: int = TILE, shared: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                  act, tile: int = TILE, shared: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
+                  identity: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Token-choice MoE for inference: ``sum_k p_k * W_down[e_k] act(W_in[e_k] h)`` -> fp32 [T, D]. Gated experts:
     ``w_gate_up`` [E, 2F, D] (gate rows first) and ``act`` maps [rows, 2F] -> [rows, F]; plain experts: ``w_gate_up`` is the
     up projection [E, F, D] and ``act`` an elementwise activation. ``w_down`` [E, D, F]. Tokens are counting-sorted by expert
     on the device (``dispatch``), both projections are one grouped GEMM each, and the weighted sum over a token's experts
-    (plus ``gate * shared``, a shared expert's rows, when given) is taken in fp32 in a fixed order (``moe_combine``)."""
+    (plus ``gate * shared``, a shared expert's rows, when given) is taken in fp32 in a fixed order (``moe_combine``).
+    Expert indices of E and above are identity experts: their output is the token's row of ``identity`` (fp32 [T, D])."""
     E = w_gate_up.shape[0]
     d = dispatch(top_i, E, tile)
-    xs = torch.zeros(d.rows, h.shape[1], dtype=h.dtype, device=h.device).index_copy(0, d.dest, h.index_select(0, d.tok))
-    mid = act(grouped_linear(xs, w_gate_up, None, d, tile))
+    mid = act(grouped_linear(gather_rows(h, d), w_gate_up, None, d, tile))
     y = grouped_linear(mid, w_down, None, d, tile)
-    return moe_combine(y.contiguous(), d.dest, top_p, shared, gate)
+    return moe_combine(y.contiguous(), d.dest, top_p, shared, gate, identity)

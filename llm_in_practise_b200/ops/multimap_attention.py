@@ -21,9 +21,11 @@ from typing import Optional
 import torch
 
 from . import _native as nv
+from .linear_scan import _conv_tail, short_conv
 
 vp, i32, i64, f32 = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong, ctypes.c_float
 _MMA_D, _MMA_DV = (32, 48, 64, 96, 128), (32, 64, 96, 128)        # sizes the tensor-core kernel is built for
+_CONV_TAPS = 5                                                     # taps of the fused convolution + norm + store
 _SPLIT_KEYS = int(os.environ.get("B200_PAGED_SPLIT_KEYS", "512"))  # keys per range of a small batch with many visible keys
 
 
@@ -72,26 +74,80 @@ def qknorm_rope_store(proj: torch.Tensor, wq: torch.Tensor, wk: Optional[torch.T
     return q_out
 
 
+def conv_qknorm_store(proj: torch.Tensor, bias: Optional[torch.Tensor], w: torch.Tensor, tail: torch.Tensor, pos: torch.Tensor,
+                      slot: torch.Tensor, runs: Optional[torch.Tensor], n_runs: int, cache_k: torch.Tensor, cache_v: torch.Tensor,
+                      table: torch.Tensor, H: int, G: int, D: int, Dv: int, eps: float, dtype: torch.dtype, temp=(0.0, 1.0),
+                      norm_qk: bool = True, norm_v: bool = False) -> torch.Tensor:
+    """Convolved queries, keys and values of one-map attention. ``proj`` [T, >= (H + G) D + G Dv] = q | k | v rows (fp32 or bf16)
+    gets ``bias`` (fp32 [C] or None), then every channel a causal convolution over time (``w`` fp32 [C, taps]; the last
+    taps - 1 biased inputs of a sequence wait in ``tail`` fp32 [rows, taps - 1, C], advanced here); then each q and k row is
+    divided by its root mean square (``norm_qk``), each v row too (``norm_v``), and q at position p is multiplied by
+    1 + c ln(floor((p + 1) / every) + 1) with ``temp`` = (c, every). Returns q [T, H * D] in ``dtype``; keys and values are
+    written at (slot, pos) of the pools."""
+    T = proj.shape[0]
+    C, taps = w.shape
+    q_out = torch.empty(T, H * D, dtype=dtype, device=proj.device)
+    BS = cache_k.shape[2]
+    if nv.use_native(proj):
+        if proj.dtype not in (torch.float32, torch.bfloat16) or proj.stride(1) != 1 or cache_k.dtype != dtype:
+            raise ValueError("conv_qknorm_store: fp32 or bf16 rows with a contiguous last dim, q in the cache dtype")
+        if taps > _CONV_TAPS:                            # more taps than the fused kernel holds in registers: convolve first
+            u = proj[:, :C].float() + bias if bias is not None else proj[:, :C]
+            proj, bias, taps = short_conv(u, w, tail, pos, slot, runs, n_runs, act=False, out_dtype=proj.dtype), None, 1
+            w = torch.ones(C, 1, dtype=torch.float32, device=proj.device)
+        fn = nv.proto("b200_conv_qknorm_store", [vp, i64, vp, vp, vp, vp, vp, vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32,
+                                                 f32, f32, i32, i32, i32, i32, vp])
+        nv.check(fn(nv.ptr(proj), proj.stride(0), nv.ptr(bias), nv.ptr(w), nv.ptr(tail), nv.ptr(pos), nv.ptr(slot), nv.ptr(table),
+                    table.shape[1], nv.ptr(q_out), nv.ptr(cache_k), nv.ptr(cache_v), T, H, G, D, Dv, taps, BS, float(eps),
+                    float(temp[0]), float(temp[1]), int(norm_qk), int(norm_v), nv.dtype_code(proj.dtype), nv.dtype_code(dtype),
+                    nv.stream()), "conv_qknorm_store")
+        nv.count_launch()
+        if taps > 1:
+            _conv_tail(proj, bias, tail, runs, pos, slot, n_runs if runs is not None else T, C, taps)
+        return q_out
+    u = proj[:, :C].float()
+    if bias is not None:
+        u = u + bias.float()
+    y = short_conv(u, w, tail, pos, slot, runs, n_runs, act=False)
+    nq, nk = H * D, G * D
+    unit = lambda x: x * torch.rsqrt((x * x).mean(-1, keepdim=True) + eps)                       # noqa: E731
+    q, k, v = y[:, :nq].view(T, H, D), y[:, nq:nq + nk].view(T, G, D), y[:, nq + nk:].reshape(T, G, Dv)
+    if norm_qk:
+        q, k = unit(q), unit(k)
+    if norm_v:
+        v = unit(v)
+    t = 1.0 + temp[0] * torch.log(torch.floor((pos.double() + 1) / temp[1]) + 1).float()
+    q_out.copy_((q * t.view(T, 1, 1)).reshape(T, nq).to(dtype))
+    pl, sl = pos.long(), slot.long()
+    blk, off = table[sl, pl // BS].long(), pl % BS
+    cache_k[blk, :, off] = k.to(cache_k.dtype)
+    cache_v[blk, :, off] = v.to(cache_v.dtype)
+    return q_out
+
+
 def multimap_attention(q: torch.Tensor, cache_k: torch.Tensor, cache_v: torch.Tensor, table: torch.Tensor, pos: torch.Tensor,
                        slot: torch.Tensor, H: int, G: int, M: int, D: int, Dv: int, scale: float, window: int = 0,
                        keep_first: int = 0, combine: bool = False, lam: float = 0.0, post: float = 1.0, eps: float = 0.0,
-                       pieces=None, max_pos: int = 0) -> torch.Tensor:
+                       pieces=None, max_pos: int = 0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Context [T, H * Dv] (q's dtype) of ``q`` [T, H * M * D] over the pools; see the module docstring for the mask and the
-    combination. ``pieces`` (``inference.ragged.Pieces``): bf16 steps with a run of 8 or more tokens go through the tensor-core
+    combination; ``post`` multiplies the result with and without it. ``out``: where to write it (rows may be strided). ``pieces`` (``inference.ragged.Pieces``): bf16 steps with a run of 8 or more tokens go through the tensor-core
     kernel; everything else (fp32, decode batches, sizes it is not built for) through the per-token kernels. ``max_pos``: an upper
     bound of ``pos`` known on the host (0 = unknown), used to cut the keys of a small batch into ranges."""
     T = q.shape[0]
     BS = cache_k.shape[2]
-    out = torch.empty(T, H * Dv, dtype=q.dtype, device=q.device)
+    if out is None:
+        out = torch.empty(T, H * Dv, dtype=q.dtype, device=q.device)
     if nv.use_native(q):
         if cache_k.dtype != q.dtype or not q.is_contiguous():
             raise ValueError("multimap_attention: contiguous q in the cache dtype")
+        if out.dtype != q.dtype or out.stride(1) != 1:
+            raise ValueError("multimap_attention: out in q's dtype with a contiguous last dim")
         if (pieces is not None and pieces.longest >= 8 and q.dtype == torch.bfloat16 and D in _MMA_D and Dv in _MMA_DV and scale > 0
-                and BS & (BS - 1) == 0 and os.environ.get("B200_PAGED_MMA", "1") != "0"):
-            fn = nv.proto("b200_multimap_attn_mma", [vp, vp, vp, vp, i32, vp, i32, vp, i32, i32, i32, i32, i32, i32, f32, i32, i32, i32,
+                and BS & (BS - 1) == 0 and out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0 and os.environ.get("B200_PAGED_MMA", "1") != "0"):
+            fn = nv.proto("b200_multimap_attn_mma", [vp, vp, vp, vp, i32, vp, i32, vp, i64, i32, i32, i32, i32, i32, i32, f32, i32, i32, i32,
                                                      f32, f32, f32, i32, vp])
             nv.check(fn(nv.ptr(q), nv.ptr(cache_k), nv.ptr(cache_v), nv.ptr(pieces.tiles), pieces.n_tiles, nv.ptr(table),
-                        table.shape[1], nv.ptr(out), H, G, M, D, Dv, BS, float(scale), int(window), int(keep_first), int(combine),
+                        table.shape[1], nv.ptr(out), out.stride(0), H, G, M, D, Dv, BS, float(scale), int(window), int(keep_first), int(combine),
                         float(lam), float(post), float(eps), nv.dtype_code(q.dtype), nv.stream()), "multimap_attn_mma")
             nv.count_launch()
             return out
@@ -103,10 +159,10 @@ def multimap_attention(q: torch.Tensor, cache_k: torch.Tensor, cache_v: torch.Te
         if seen > 2 * _SPLIT_KEYS and T * G < 296:
             nsplit = min(32, -(-seen // _SPLIT_KEYS), max(1, 592 // (T * G)))
         part = torch.empty(T * H * M * nsplit * (Dv + 2), dtype=torch.float32, device=q.device) if nsplit * M > 1 else None
-        fn = nv.proto("b200_multimap_attn", [vp, vp, vp, vp, vp, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, i32, i32,
+        fn = nv.proto("b200_multimap_attn", [vp, vp, vp, vp, vp, vp, i32, vp, i64, vp, i32, i32, i32, i32, i32, i32, i32, f32, i32, i32,
                                              i32, i32, f32, f32, f32, i32, vp])
         nv.check(fn(nv.ptr(q), nv.ptr(cache_k), nv.ptr(cache_v), nv.ptr(pos), nv.ptr(slot), nv.ptr(table), table.shape[1],
-                    nv.ptr(out), nv.ptr(part), T, H, G, M, D, Dv, BS, float(scale), int(window), int(keep_first), nsplit, int(combine),
+                    nv.ptr(out), out.stride(0), nv.ptr(part), T, H, G, M, D, Dv, BS, float(scale), int(window), int(keep_first), nsplit, int(combine),
                     float(lam), float(post), float(eps), nv.dtype_code(q.dtype), nv.stream()), "multimap_attn")
         nv.count_launch(2 if nsplit * M > 1 else 1)
         return out
@@ -126,6 +182,7 @@ def multimap_attention(q: torch.Tensor, cache_k: torch.Tensor, cache_v: torch.Te
         a = torch.einsum("hmn,nhe->hme", sc.softmax(-1), v)
         o = a[:, 0] - lam * a[:, 1] if M == 2 else a[:, 0]
         if combine:
-            o = o * torch.rsqrt((o * o).mean(-1, keepdim=True) + eps) * post
+            o = o * torch.rsqrt((o * o).mean(-1, keepdim=True) + eps)
+        o = o * post
         out[t] = o.reshape(H * Dv).to(q.dtype)
     return out

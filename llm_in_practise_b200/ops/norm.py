@@ -200,3 +200,20 @@ def sandwich_norm(y: Optional[torch.Tensor], post_w: Optional[torch.Tensor], res
     elif cast_next:
         h = x.to(out_dtype)
     return h, x
+
+
+def poly_norm(z: torch.Tensor, act: torch.Tensor, eps: float) -> torch.Tensor:
+    """``a N(z) + b N(z^2) + c N(z^3) + e`` per row of ``z`` [T, F], powers element by element, N(y) = y / sqrt(mean(y^2) + eps)
+    over the row, ``act`` = (a, b, c, e) fp32 [4]. fp32 arithmetic, output in z's dtype. Inference only."""
+    rows, cols = z.shape
+    if nv.use_native(z):
+        z = z.contiguous()
+        y = torch.empty_like(z)
+        fn = nv.proto("b200_poly_norm", [vp, vp, vp, i64, i32, f32, i32, vp])
+        nv.check(fn(nv.ptr(z), nv.ptr(act), nv.ptr(y), rows, cols, float(eps), nv.dtype_code(z.dtype), nv.stream()), "poly_norm")
+        nv.count_launch()
+        return y
+    zf = z.float()
+    unit = lambda v: v / torch.sqrt((v * v).mean(-1, keepdim=True) + eps)                        # noqa: E731
+    a = act.float()
+    return (a[0] * unit(zf) + a[1] * unit(zf * zf) + a[2] * unit(zf * zf * zf) + a[3]).to(z.dtype)

@@ -124,6 +124,9 @@ class LLMEngine:
         if gen_cls is Generator and getattr(getattr(model, "base_model", model), "ragged", False):
             from ..inference.ragged import RaggedGenerator
             gen_cls = RaggedGenerator                    # models served by one ragged step (prompt pieces + decode tokens mixed)
+        limit = getattr(getattr(model, "base_model", model), "max_positions", 0)
+        if limit:                                        # a learned position table: no row can be longer
+            self.args.max_model_len = min(self.args.max_model_len, int(limit))
         self.gen = gen_cls(model, tokenizer, self.args.max_model_len)
         self.model, self.tokenizer, self.model_name = self.gen.model, tokenizer, model_name
         self.ragged = bool(getattr(self.gen, "ragged", False))
