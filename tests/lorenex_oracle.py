@@ -32,14 +32,11 @@ def causal_conv(u, w, bias=None):
     n, C = u.shape
     taps = w.shape[1]
     y = torch.zeros(n, C, dtype=F64)
-    for t in range(n):
-        for j in range(taps):
-            s = t - taps + 1 + j
-            if s >= 0:
-                y[t] += w[:, j].to(F64) * u[s]
-        if bias is not None:
-            y[t] += bias.to(F64)
-    return y
+    for j in range(taps):
+        back = taps - 1 - j                        # w[:, j] weighs the input `back` tokens ago
+        if back < n:
+            y[back:] += w[:, j].to(F64) * u[:n - back]
+    return y if bias is None else y + bias.to(F64)
 
 
 def gla_decay(z, tau):
