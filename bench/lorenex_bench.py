@@ -194,7 +194,7 @@ def kernel_rows(size, dev, steps, warmup, root):
     del ckd, cvd
     # --- decays of the matrix memory vs Duratar's gates
     a1, a2, ab = rnd(T, rank), rnd(SH * SD, rank), torch.full((SH * SD,), 2.0, device=dev)
-    ms_k = t(lambda: lowrank_decay(a1, a2, ab, 16.0), steps, warmup)
+    ms_k = t(lambda: lowrank_decay(a1, a2, ab, 16.0, fast=True), steps, warmup)
     SG = max(1, SH // 4)
     qs, ks, aa, bb = rnd(T, SG * SD), rnd(T, SG * SD), rnd(T, SH * SD), rnd(T, SH)
     dtb, alog = torch.zeros(SH * SD, device=dev), torch.zeros(SH, device=dev)
@@ -202,7 +202,7 @@ def kernel_rows(size, dev, steps, warmup, root):
     rows.append((f"per-channel decays from a rank-{rank} input, {SH * SD} channels", ms_k, frac_bw(T * SH * SD * 4, ms_k),
                  "Duratar: unit q / k, decays, beta", ms_l, frac_bw(T * (2 * SG * SD + SH * SD + SH) * 8, ms_l), "HBM"))
     # --- matrix memory: prompt and decode batch
-    g = lowrank_decay(a1, a2, ab, 16.0)
+    g = lowrank_decay(a1, a2, ab, 16.0, fast=True)
     q16, k16, vs = rnd(T, SH * SD) * SD ** -0.5, rnd(T, SH * SD) * SD ** -0.5, rnd(T, SH * SDv)
     st0 = torch.zeros(Bq + 1, SH, SD, SDv, device=dev)
     ga, gb = torch.rand(T, SH, device=dev) * 0.1 + 0.9, torch.rand(T, SH, device=dev)

@@ -304,8 +304,12 @@ channel_scan_carry_kernel(float* __restrict__ part, const float* __restrict__ pd
   }
 }
 
-// One thread per channel and kTok tokens: the channel's weights are read once; x rows are broadcast from shared memory.
-constexpr int kLrTok = 8;
+// One thread per channel and kLrTok tokens: the channel's weights are read once; x rows are broadcast from shared memory.
+// FAST (16-bit models): base-2 hardware exponential and logarithm; their absolute error in log sigmoid, 2e-7, is divided by tau.
+// Otherwise a decay near 1 is formed as 1 + expm1(.): it is raised to the power of its whole reach, and expf's small bias would
+// add up where the rounding of 1 + expm1 does not.
+constexpr int kLrTok = 16;
+template <bool FAST>
 __global__ void __launch_bounds__(128)
 lowrank_decay_kernel(const float* __restrict__ x, long long ldx, const float* __restrict__ w2, const float* __restrict__ bias,
                      float* __restrict__ out, int tokens, int C, int rank, float inv_tau) {
@@ -347,22 +351,29 @@ lowrank_decay_kernel(const float* __restrict__ x, long long ldx, const float* __
   for (int t = 0; t < kLrTok; ++t) {
     if (t >= nt) break;
     const float z = acc[t];
-    const float ls = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));        // log sigmoid(z)
-    // a decay near 1 is raised to the power of its whole reach: 1 + expm1 rounds once, without expf's small bias
-    out[(long long)(t0 + t) * C + c] = 1.f + expm1f(ls * inv_tau);
+    float v;
+    if (FAST) {
+      const float z2 = z * 1.4426950408889634f;
+      v = exp2f((fminf(z2, 0.f) - __log2f(1.f + exp2f(-fabsf(z2)))) * inv_tau);
+    } else {
+      const float y = (fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * inv_tau;        // log sigmoid(z) / tau
+      v = y > -0.5f ? 1.f + expm1f(y) : expf(y);
+    }
+    out[(long long)(t0 + t) * C + c] = v;
   }
 }
 }  // namespace b200
 
 B200_API int b200_lowrank_decay(const float* x, long long ldx, const float* w2, const float* bias, float* out, int tokens, int C,
-                                int rank, float inv_tau, void* stream) {
+                                int rank, float inv_tau, int fast, void* stream) {
   using namespace b200;
   if (tokens <= 0) return 0;
   if (C <= 0 || rank <= 0 || tokens > 65535 * kLrTok) return B200_ERR_BAD_SHAPE;
   const size_t smem = (size_t)kLrTok * rank * 4;
   if (smem > 48 * 1024) return B200_ERR_TOO_LARGE;
   dim3 grid((C + 127) / 128, (tokens + kLrTok - 1) / kLrTok);
-  lowrank_decay_kernel<<<grid, 128, smem, (cudaStream_t)stream>>>(x, ldx, w2, bias, out, tokens, C, rank, inv_tau);
+  if (fast) lowrank_decay_kernel<true><<<grid, 128, smem, (cudaStream_t)stream>>>(x, ldx, w2, bias, out, tokens, C, rank, inv_tau);
+  else lowrank_decay_kernel<false><<<grid, 128, smem, (cudaStream_t)stream>>>(x, ldx, w2, bias, out, tokens, C, rank, inv_tau);
   B200_LAUNCH_CHECK();
   return 0;
 }

@@ -93,10 +93,72 @@ __global__ void short_conv_kernel(const TX* __restrict__ x, long long ldx, const
   for (int e = 0; e < V; ++e) acc[e] = (act ? silu_f(acc[e]) : acc[e]) + (residual ? own[e] : 0.f);
   TY* dst = y + (long long)t * ldy + c;
   if (V == 4 && sizeof(TY) == 4) *reinterpret_cast<float4*>(dst) = *reinterpret_cast<const float4*>(acc);
-  else if (V == 4) *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16x2(acc[0], acc[1]), pack_bf16x2(acc[V - 2], acc[V - 1]));
+  else if (V == 4) *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16x2(acc[0], acc[1 % V]), pack_bf16x2(acc[V - 2 >= 0 ? V - 2 : 0], acc[V - 1]));
   else {
 #pragma unroll
     for (int e = 0; e < V; ++e) dst[e] = from_f32<TY>(acc[e]);
+  }
+}
+
+// The same over prompt pieces, for few taps: a thread owns V channels over TB consecutive tokens, keeps their weights and last
+// TAPS - 1 inputs in registers, and fetches what lies before a token only where a run starts (from x, the tail, or zeros).
+template <int V, typename TX, typename TY, int TAPS>
+__global__ void __launch_bounds__(128)
+short_conv_run_kernel(const TX* __restrict__ x, long long ldx, const float* __restrict__ w, const float* __restrict__ bias,
+                      const float* __restrict__ state, const int* __restrict__ pos, const int* __restrict__ slot, TY* __restrict__ y,
+                      long long ldy, int tokens, int C, int act, int residual, int TB) {
+  constexpr int L = TAPS - 1, LH = L > 0 ? L : 1;
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+  if (c >= C) return;
+  float wt[TAPS][V], hist[LH][V], b[V];
+#pragma unroll
+  for (int e = 0; e < V; ++e) {
+    b[e] = bias ? bias[c + e] : 0.f;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) wt[j][e] = w[(long long)(c + e) * TAPS + j];
+#pragma unroll
+    for (int j = 0; j < LH; ++j) hist[j][e] = 0.f;
+  }
+  const int t0 = blockIdx.y * TB, t1 = min(tokens, t0 + TB);
+  int ps = -1, pp = -2;
+#pragma unroll 4
+  for (int t = t0; t < t1; ++t) {
+    const int p = pos[t], s = slot[t];
+    if (L > 0 && !(s == ps && p == pp + 1)) {
+      int nb = 0;
+      while (nb < L && t - nb - 1 >= 0 && slot[t - nb - 1] == s && pos[t - nb - 1] == p - nb - 1) ++nb;
+#pragma unroll
+      for (int d = 1; d <= L; ++d) {                       // d tokens back -> hist[L - d]
+        float v[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[e] = 0.f;
+        if (p - d >= 0) {
+          if (d <= nb) load_f32<V, TX>(x + (long long)(t - d) * ldx + c, v);
+          else load_f32<V, float>(state + ((long long)s * L + (L - (d - nb))) * C + c, v);
+        }
+#pragma unroll
+        for (int e = 0; e < V; ++e) hist[L > 0 ? L - d : 0][e] = v[e];
+      }
+    }
+    ps = s; pp = p;
+    float v[V], a[V];
+    load_f32<V, TX>(x + (long long)t * ldx + c, v);
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      float acc = b[e];
+#pragma unroll
+      for (int j = 0; j < L; ++j) acc = fmaf(wt[j][e], hist[j][e], acc);
+      acc = fmaf(wt[TAPS - 1][e], v[e], acc);
+#pragma unroll
+      for (int j = 0; j + 1 < L; ++j) hist[j][e] = hist[j + 1][e];
+      if (L > 0) hist[LH - 1][e] = v[e];
+      if (act) acc = sizeof(TY) == 4 ? silu_f(acc) : __fdividef(acc, 1.f + __expf(-acc));
+      a[e] = acc + (residual ? v[e] : 0.f);
+    }
+    TY* dst = y + (long long)t * ldy + c;
+    if (V == 4 && sizeof(TY) == 4) *reinterpret_cast<float4*>(dst) = *reinterpret_cast<const float4*>(a);
+    else if (V == 4) *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16x2(a[0], a[1 % V]), pack_bf16x2(a[V - 2 >= 0 ? V - 2 : 0], a[V - 1]));
+    else dst[0] = from_f32<TY>(a[0]);
   }
 }
 
@@ -539,6 +601,28 @@ B200_API int b200_short_conv_ex(const void* x, long long ldx, const float* w, co
                    !(reinterpret_cast<uintptr_t>(y) & (y_dtype == B200_DT_FP32 ? 15 : 7));
   const long long n = (long long)tokens * (vec ? C / 4 : C);
   const unsigned grid = (unsigned)((n + 255) / 256);
+  if (!step_tail && taps <= 5) {
+    const int TB = tokens >= 2048 ? 16 : (tokens >= 256 ? 4 : 1);
+    const int per = 128 * (vec ? 4 : 1);
+    const dim3 rgrid((C + per - 1) / per, (tokens + TB - 1) / TB);
+    if (rgrid.y > 65535) return B200_ERR_TOO_LARGE;
+#define CONVR(VV, TX, TY, TT)                                                                                                \
+  short_conv_run_kernel<VV, TX, TY, TT><<<rgrid, 128, 0, st>>>((const TX*)x, ldx, w, bias, state, pos, slot, (TY*)y, ldy, tokens, C, act, \
+                                                               residual, TB)
+#define CONVR_T(VV, TX, TY)                                                                                                  \
+  switch (taps) {                                                                                                            \
+    case 1: CONVR(VV, TX, TY, 1); break; case 2: CONVR(VV, TX, TY, 2); break; case 3: CONVR(VV, TX, TY, 3); break;           \
+    case 4: CONVR(VV, TX, TY, 4); break; default: CONVR(VV, TX, TY, 5); break;                                               \
+  }
+#define CONVR_Y(TX, TY) do { if (vec) { CONVR_T(4, TX, TY) } else { CONVR_T(1, TX, TY) } } while (0)
+    if (x_dtype == B200_DT_FP32) { if (y_dtype == B200_DT_FP32) CONVR_Y(float, float); else CONVR_Y(float, __nv_bfloat16); }
+    else { if (y_dtype == B200_DT_FP32) CONVR_Y(__nv_bfloat16, float); else CONVR_Y(__nv_bfloat16, __nv_bfloat16); }
+#undef CONVR_Y
+#undef CONVR_T
+#undef CONVR
+    B200_LAUNCH_CHECK();
+    return 0;
+  }
 #define CONV(VV, TX, TY)                                                                                                     \
   short_conv_kernel<VV, TX, TY><<<grid, 256, 0, st>>>((const TX*)x, ldx, w, bias, state, pos, slot, (TY*)y, ldy, tokens, C, taps, act, \
                                                       residual, step_tail)

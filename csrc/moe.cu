@@ -132,18 +132,21 @@ moe_route_grouped_kernel(const TH* __restrict__ h, const TW* __restrict__ wr, co
   const TH* hr = h + t * W;
   route_logits<TH, TW>(hr, wr, W, E + X, lane, s);
   __syncwarp();
-  if (lane != 0) return;
-  for (int e = softmax ? E : 0; e < E + X; ++e) s[e] = 1.f / (1.f + expf(-s[e]));
+  for (int e = (softmax ? E : 0) + lane; e < E + X; e += 32) s[e] = 1.f / (1.f + expf(-s[e]));
   if (softmax) {                                       // scores are the softmax of the logits over all experts
     float zmax = -INFINITY, zsum = 0.f;
-    for (int e = 0; e < E; ++e) zmax = fmaxf(zmax, s[e]);
-    for (int e = 0; e < E; ++e) { s[e] = expf(s[e] - zmax); zsum += s[e]; }
-    for (int e = 0; e < E; ++e) s[e] /= zsum;
+    for (int e = lane; e < E; e += 32) zmax = fmaxf(zmax, s[e]);
+    zmax = warp_max(zmax);
+    for (int e = lane; e < E; e += 32) { s[e] = expf(s[e] - zmax); zsum += s[e]; }
+    zsum = warp_sum(zsum);
+    for (int e = lane; e < E; e += 32) s[e] /= zsum;
   }
-  for (int x = 0; x < X; ++x) gate_out[t * X + x] = s[E + x];
-  for (int e = 0; e < E; ++e) choice[e] = s[e] + (corr ? corr[e] : 0.f);
+  __syncwarp();
+  for (int x = lane; x < X; x += 32) gate_out[t * X + x] = s[E + x];
+  for (int e = lane; e < E; e += 32) choice[e] = s[e] + (corr ? corr[e] : 0.f);
+  __syncwarp();
   const int per = E / groups;
-  if (keep < groups) {
+  if (keep < groups && lane == 0) {
     for (int g = 0; g < groups; ++g) {                 // sum of the group's `group_top` largest choice scores
       float sum = 0.f;
       int last = -1;
@@ -173,18 +176,28 @@ moe_route_grouped_kernel(const TH* __restrict__ h, const TW* __restrict__ wr, co
     for (int e = 0; e < E; ++e)
       if (gs[e / per] != INFINITY) choice[e] = -INFINITY;
   }
+  __syncwarp();
   float psum = 0.f;
-  for (int k = 0; k < top; ++k) {
-    int best = 0;
-    float bv = choice[0];
-    for (int e = 1; e < E; ++e)
-      if (choice[e] > bv) { best = e; bv = choice[e]; }
-    choice[best] = -INFINITY;                          // taken
-    top_i[t * top + k] = best;
-    top_p[t * top + k] = s[best];
+  for (int k = 0; k < top; ++k) {                      // the largest choice score left, the lower index among equals
+    int best = E;
+    float bv = -INFINITY;
+    for (int e = lane; e < E; e += 32)
+      if (choice[e] > bv || best == E) { best = e; bv = choice[e]; }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float v2 = __shfl_xor_sync(0xffffffffu, bv, o);
+      const int b2 = __shfl_xor_sync(0xffffffffu, best, o);
+      if (v2 > bv || (v2 == bv && b2 < best)) { bv = v2; best = b2; }
+    }
+    if (lane == 0) {
+      choice[best] = -INFINITY;                        // taken
+      top_i[t * top + k] = best;
+      top_p[t * top + k] = s[best];
+    }
     psum += s[best];
+    __syncwarp();
   }
-  if (renorm)
+  if (renorm && lane == 0)
     for (int k = 0; k < top; ++k) top_p[t * top + k] /= psum;
 }
 

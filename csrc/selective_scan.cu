@@ -33,20 +33,21 @@ struct SelScanArgs {
   int n_tiles, inner, N, chunk;
 };
 
-// PASS 0: blockIdx.x is a run; 1, 2: a tile
+__device__ __forceinline__ float decay_exact(float x) { return x > -0.5f ? 1.f + expm1f(x) : expf(x); }
+
+// PASS 0: blockIdx.x is a run, 3: a token (a decode batch); 1, 2: a tile
 template <typename T, int R, int LPC, int PASS>
 __global__ void __launch_bounds__(128)
 selective_scan_kernel(const SelScanArgs a) {
   extern __shared__ __align__(16) float sm[];            // [chunk][B: NP | C: NP]
   constexpr bool exact = sizeof(T) == 4;
-  constexpr int NP = R * LPC, cpw = 32 / LPC, U = 4;
+  constexpr int NP = R * LPC, cpw = 32 / LPC, U = PASS == 3 ? 1 : 4;
   const int b_ = blockIdx.x;
   int first, n, p0, s;
   bool last_tile = true;
-  if (PASS == 0) {
-    if (a.runs) { first = a.runs[4 * b_]; n = a.runs[4 * b_ + 1]; p0 = a.runs[4 * b_ + 2]; s = a.runs[4 * b_ + 3]; }
-    else { first = b_; n = 1; p0 = a.pos[b_]; s = a.slot[b_]; }
-  } else {
+  if (PASS == 0) { first = a.runs[4 * b_]; n = a.runs[4 * b_ + 1]; p0 = a.runs[4 * b_ + 2]; s = a.runs[4 * b_ + 3]; }
+  else if (PASS == 3) { first = b_; n = 1; p0 = a.pos[b_]; s = a.slot[b_]; }
+  else {
     last_tile = a.tile_of[4 * b_ + 1] + 1 == a.tile_of[4 * b_ + 2];
     if (PASS == 1 && last_tile) return;
     first = a.tiles[4 * b_]; n = a.tiles[4 * b_ + 1]; p0 = a.tiles[4 * b_ + 2]; s = a.tiles[4 * b_ + 3];
@@ -60,8 +61,8 @@ selective_scan_kernel(const SelScanArgs a) {
   const int n0 = l * R;
   float2 S2[R / 2], A2[R / 2];
   float* sp = a.state + (long long)s * N * inner + cl;
-  float* pp = PASS == 0 ? nullptr : a.part + (long long)b_ * N * inner + cl;
-  const float* src = PASS == 2 ? pp : (PASS == 0 && p0 > 0 ? sp : nullptr);
+  float* pp = PASS == 0 || PASS == 3 ? nullptr : a.part + (long long)b_ * N * inner + cl;
+  const float* src = PASS == 2 ? pp : (PASS != 1 && p0 > 0 ? sp : nullptr);
 #pragma unroll
   for (int i = 0; i < R / 2; ++i) {
     float av[2], sv[2];
@@ -127,8 +128,8 @@ selective_scan_kernel(const SelScanArgs a) {
           const float4 b4 = *reinterpret_cast<const float4*>(bs + 2 * i);
           float2 xa = __fmul2_rn(A2[i], s2), xb = __fmul2_rn(A2[i + 1], s2);
           if (exact) {
-            xa = make_float2(1.f + expm1f(xa.x), 1.f + expm1f(xa.y));
-            xb = make_float2(1.f + expm1f(xb.x), 1.f + expm1f(xb.y));
+            xa = make_float2(decay_exact(xa.x), decay_exact(xa.y));
+            xb = make_float2(decay_exact(xb.x), decay_exact(xb.y));
           } else {
             xa = make_float2(ex2_approx(xa.x), ex2_approx(xa.y));
             xb = make_float2(ex2_approx(xb.x), ex2_approx(xb.y));
@@ -204,7 +205,9 @@ static int sel_launch(const SelScanArgs& a, int n_runs, cudaStream_t st) {
     if (smem > 48 * 1024) B200_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));  \
     kern<<<dim3(NB, cb), 128, smem, st>>>(a);                                                                              \
   } while (0)
-  if (a.n_tiles <= 0) {
+  if (!a.runs) {
+    SEL(3, n_runs);
+  } else if (a.n_tiles <= 0) {
     SEL(0, n_runs);
   } else {
     SEL(1, a.n_tiles);

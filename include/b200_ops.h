@@ -636,12 +636,12 @@ int b200_scan_readout(const float* o, int ocols, const float* e, float den_eps, 
                       const float* w, int w_full, void* out, long long tokens, int H, int Dv, int groups, float eps, int out_dtype, void* stream);
 
 /* Per-channel decays of a low-rank input and the scan that uses them (csrc/channel_scan.cu): out[t, c] = sigmoid(w2[c] . x[t] +
- * bias[c])^inv_tau; per head S <- diag(g) S + k v^T, o = S^T q (fp32). n_tiles > 0: runs are walked tile by tile in parallel,
+ * bias[c])^inv_tau (fast 1: hardware exponential and logarithm); per head S <- diag(g) S + k v^T, o = S^T q (fp32). n_tiles > 0: runs are walked tile by tile in parallel,
  * tiles int32 [n_tiles, 4] = (first row, rows, first position, state row), tile_of [n_tiles, 4] = (run, place in the run, tiles
  * of the run, its first tile), run_tiles [n_runs, 4] = (first tile, tiles, 0, 0), part fp32 [n_tiles, H, D, Dv] and pdec fp32
  * [n_tiles, H, D] are scratch. chunk: tokens staged at a time (at most 16). */
 int b200_lowrank_decay(const float* x, long long ldx, const float* w2, const float* bias, float* out, int tokens, int C, int rank,
-                       float inv_tau, void* stream);
+                       float inv_tau, int fast, void* stream);
 int b200_channel_scan(const float* q, long long ldq, const float* k, long long ldk, const float* v, long long ldv, const float* g,
                       long long ldg, float* state, float* part, float* pdec, const int* runs, int n_runs, const int* tiles,
                       int n_tiles, const int* tile_of, const int* run_tiles, int chunk, const int* pos, const int* slot, float* o,

@@ -230,7 +230,7 @@ class LorenexLayer(nn.Module):
         H, D, Dv = m.heads, m.dim, m.vdim
         proj = linear_exact(h, self.in_proj, out_dtype=torch.float32)
         sl = lambda n: proj[:, self.parts[n][0]:self.parts[n][1]]             # noqa: E731
-        a = lowrank_decay(sl("a1"), self.a2, self.a2_bias, m.tau)
+        a = lowrank_decay(sl("a1"), self.a2, self.a2_bias, m.tau, fast=h.dtype != torch.float32)
         runs, n_runs = (pieces.runs, pieces.n_runs) if pieces is not None else (None, h.shape[0])
         o = linear_scan(sl("q"), sl("k"), sl("v"), state[0], pos, slot, runs, n_runs, H, H, D, Dv, "channel", g=a, pieces=pieces)
         # the queries' 1 / sqrt(dim) is a factor of o: it is applied where the heads are normed

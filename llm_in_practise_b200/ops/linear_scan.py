@@ -275,17 +275,17 @@ def scan_readout(o: torch.Tensor, H: int, Dv: int, w: torch.Tensor, groups: int,
     return v.to(out_dtype)
 
 
-def lowrank_decay(x: torch.Tensor, w2: torch.Tensor, bias: torch.Tensor, tau: float) -> torch.Tensor:
+def lowrank_decay(x: torch.Tensor, w2: torch.Tensor, bias: torch.Tensor, tau: float, fast: bool = False) -> torch.Tensor:
     """``x`` fp32 [T, r] (rows may be strided), ``w2`` fp32 [C, r], ``bias`` fp32 [C] -> sigmoid(w2 x + bias)^(1 / tau), fp32
-    [T, C], formed as exp(log sigmoid(.) / tau)."""
+    [T, C], formed as exp(log sigmoid(.) / tau). ``fast``: with the hardware's exponential and logarithm (models in 16 bits)."""
     T, r = x.shape
     C = w2.shape[0]
     if nv.use_native(x):
         if x.dtype != torch.float32 or x.stride(1) != 1:
             raise ValueError("lowrank_decay: fp32 rows with a contiguous last dim")
         out = torch.empty(T, C, dtype=torch.float32, device=x.device)
-        fn = nv.proto("b200_lowrank_decay", [vp, i64, vp, vp, vp, i32, i32, i32, f32, vp])
-        nv.check(fn(nv.ptr(x), x.stride(0), nv.ptr(w2), nv.ptr(bias), nv.ptr(out), T, C, r, 1.0 / float(tau), nv.stream()), "lowrank_decay")
+        fn = nv.proto("b200_lowrank_decay", [vp, i64, vp, vp, vp, i32, i32, i32, f32, i32, vp])
+        nv.check(fn(nv.ptr(x), x.stride(0), nv.ptr(w2), nv.ptr(bias), nv.ptr(out), T, C, r, 1.0 / float(tau), int(fast), nv.stream()), "lowrank_decay")
         nv.count_launch()
         return out
     z = x.float() @ w2.float().t() + bias.float()

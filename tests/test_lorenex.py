@@ -157,9 +157,11 @@ def test_lowrank_decay(device, dtype, C, rank, tau):
     n = 19
     buf = torch.randn(n, rank + 3, generator=g)
     w, b = torch.randn(C, rank, generator=g) * 3, torch.randn(C, generator=g) * 8          # far into both tails of the sigmoid
+    fast = lowrank_decay(buf.to(device)[:, 3:], w.to(device), b.to(device), tau, fast=True)
     got = lowrank_decay(buf.to(device)[:, 3:], w.to(device), b.to(device), tau)
     want = O.gla_decay(buf[:, 3:].double() @ w.double().T + b.double(), tau)
     torch.testing.assert_close(got.cpu().double(), want, rtol=2e-5, atol=1e-12)
+    torch.testing.assert_close(fast.cpu().double(), want, rtol=1e-4, atol=3e-7)
 
 
 def _cut_runs(lens, plans, rows):
