@@ -16,6 +16,7 @@
 // output by shuffles (each step halves the columns a lane still carries), a CTA owns a block of columns of one (run or tile,
 // head). k, q, g and v of a chunk of tokens are staged through shared memory by cp.async, one chunk ahead.
 #include "common.cuh"
+#include "mma_sync.cuh"
 #include "../include/b200_ops.h"
 
 namespace b200 {
@@ -304,62 +305,103 @@ channel_scan_carry_kernel(float* __restrict__ part, const float* __restrict__ pd
   }
 }
 
-// One thread per channel and kLrTok tokens: the channel's weights are read once; x rows are broadcast from shared memory.
+// CPT channels per thread, kLrTok tokens at a time, `groups` times: x rows of all of them are staged once and broadcast.
 // FAST (16-bit models): base-2 hardware exponential and logarithm; their absolute error in log sigmoid, 2e-7, is divided by tau.
 // Otherwise a decay near 1 is formed as 1 + expm1(.): it is raised to the power of its whole reach, and expf's small bias would
 // add up where the rounding of 1 + expm1 does not.
-constexpr int kLrTok = 16;
-template <bool FAST>
+constexpr int kLrTok = 8;
+// CPT channels per thread share the reads of x. RK: the rank at compile time, weights then stay in registers (0: any rank)
+template <bool FAST, int CPT, int RK>
 __global__ void __launch_bounds__(128)
 lowrank_decay_kernel(const float* __restrict__ x, long long ldx, const float* __restrict__ w2, const float* __restrict__ bias,
-                     float* __restrict__ out, int tokens, int C, int rank, float inv_tau) {
-  extern __shared__ __align__(16) float xs[];            // [kLrTok][rank]
-  const int t0 = blockIdx.y * kLrTok;
-  const int nt = min(kLrTok, tokens - t0);
-  for (int i = threadIdx.x; i < kLrTok * rank; i += blockDim.x) {
+                     float* __restrict__ out, int tokens, int C, int rank, float inv_tau, int groups) {
+  extern __shared__ __align__(16) float xall[];          // [groups * kLrTok][rank]
+  const int tb = blockIdx.y * kLrTok * groups;
+  for (int i = threadIdx.x; i < groups * kLrTok * rank; i += blockDim.x) {
     const int t = i / rank;
-    xs[i] = t < nt ? x[(long long)(t0 + t) * ldx + i % rank] : 0.f;
+    xall[i] = tb + t < tokens ? x[(long long)(tb + t) * ldx + i % rank] : 0.f;
   }
   __syncthreads();
-  const int c = blockIdx.x * blockDim.x + threadIdx.x;
-  if (c >= C) return;
-  float acc[kLrTok];
-  const float b = bias[c];
+  const int c0 = blockIdx.x * 128 * CPT + threadIdx.x;   // this thread's channels are 128 apart
+  const float* w[CPT];
 #pragma unroll
-  for (int t = 0; t < kLrTok; ++t) acc[t] = b;
-  const float* w = w2 + (long long)c * rank;
-  int r = 0;
-  if (rank % 4 == 0 && (reinterpret_cast<uintptr_t>(w2) & 15) == 0) {
-    for (; r < rank; r += 4) {
-      const float4 wv = *reinterpret_cast<const float4*>(w + r);
+  for (int j = 0; j < CPT; ++j) w[j] = w2 + (long long)min(c0 + 128 * j, C - 1) * rank;
+  const bool vec = rank % 4 == 0 && (reinterpret_cast<uintptr_t>(w2) & 15) == 0;
+  constexpr int RV = RK / 4 > 0 ? RK / 4 : 1;
+  float4 wr[CPT][RV];
+  if (RK > 0) {
 #pragma unroll
-      for (int t = 0; t < kLrTok; ++t) {
-        const float4 xv = *reinterpret_cast<const float4*>(xs + t * rank + r);
-        acc[t] = fmaf(wv.x, xv.x, acc[t]);
-        acc[t] = fmaf(wv.y, xv.y, acc[t]);
-        acc[t] = fmaf(wv.z, xv.z, acc[t]);
-        acc[t] = fmaf(wv.w, xv.w, acc[t]);
+    for (int j = 0; j < CPT; ++j)
+#pragma unroll
+      for (int i = 0; i < RV; ++i) wr[j][i] = *reinterpret_cast<const float4*>(w[j] + 4 * i);
+  }
+  for (int gi = 0; gi < groups; ++gi) {
+    const int t0 = tb + gi * kLrTok, nt = min(kLrTok, tokens - t0);
+    if (nt <= 0) break;
+    const float* xs = xall + gi * kLrTok * rank;
+    float acc[kLrTok][CPT];
+#pragma unroll
+    for (int j = 0; j < CPT; ++j) {
+      const float b = bias[min(c0 + 128 * j, C - 1)];
+#pragma unroll
+      for (int t = 0; t < kLrTok; ++t) acc[t][j] = b;
+    }
+    int r = RK;
+    if (RK > 0) {
+#pragma unroll
+      for (int i = 0; i < RV; ++i)
+#pragma unroll
+        for (int t = 0; t < kLrTok; ++t) {
+          const float4 xv = *reinterpret_cast<const float4*>(xs + t * rank + 4 * i);
+#pragma unroll
+          for (int j = 0; j < CPT; ++j) {
+            acc[t][j] = fmaf(wr[j][i].x, xv.x, acc[t][j]);
+            acc[t][j] = fmaf(wr[j][i].y, xv.y, acc[t][j]);
+            acc[t][j] = fmaf(wr[j][i].z, xv.z, acc[t][j]);
+            acc[t][j] = fmaf(wr[j][i].w, xv.w, acc[t][j]);
+          }
+        }
+    } else if (vec) {
+      for (; r < rank; r += 4) {
+        float4 wv[CPT];
+#pragma unroll
+        for (int j = 0; j < CPT; ++j) wv[j] = *reinterpret_cast<const float4*>(w[j] + r);
+#pragma unroll
+        for (int t = 0; t < kLrTok; ++t) {
+          const float4 xv = *reinterpret_cast<const float4*>(xs + t * rank + r);
+#pragma unroll
+          for (int j = 0; j < CPT; ++j) {
+            acc[t][j] = fmaf(wv[j].x, xv.x, acc[t][j]);
+            acc[t][j] = fmaf(wv[j].y, xv.y, acc[t][j]);
+            acc[t][j] = fmaf(wv[j].z, xv.z, acc[t][j]);
+            acc[t][j] = fmaf(wv[j].w, xv.w, acc[t][j]);
+          }
+        }
       }
     }
-  }
-  for (; r < rank; ++r) {
-    const float wv = w[r];
+    for (; r < rank; ++r) {
 #pragma unroll
-    for (int t = 0; t < kLrTok; ++t) acc[t] = fmaf(wv, xs[t * rank + r], acc[t]);
-  }
+      for (int t = 0; t < kLrTok; ++t)
 #pragma unroll
-  for (int t = 0; t < kLrTok; ++t) {
-    if (t >= nt) break;
-    const float z = acc[t];
-    float v;
-    if (FAST) {
-      const float z2 = z * 1.4426950408889634f;
-      v = exp2f((fminf(z2, 0.f) - __log2f(1.f + exp2f(-fabsf(z2)))) * inv_tau);
-    } else {
-      const float y = (fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * inv_tau;        // log sigmoid(z) / tau
-      v = y > -0.5f ? 1.f + expm1f(y) : expf(y);
+        for (int j = 0; j < CPT; ++j) acc[t][j] = fmaf(w[j][r], xs[t * rank + r], acc[t][j]);
     }
-    out[(long long)(t0 + t) * C + c] = v;
+#pragma unroll
+    for (int t = 0; t < kLrTok; ++t) {
+      if (t >= nt) break;
+#pragma unroll
+      for (int j = 0; j < CPT; ++j) {
+        const float z = acc[t][j];
+        float v;
+        if (FAST) {
+          const float z2 = z * 1.4426950408889634f;
+          v = ex2_approx((fminf(z2, 0.f) - __log2f(1.f + ex2_approx(-fabsf(z2)))) * inv_tau);
+        } else {
+          const float y = (fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * inv_tau;        // log sigmoid(z) / tau
+          v = y > -0.5f ? 1.f + expm1f(y) : expf(y);
+        }
+        if (c0 + 128 * j < C) out[(long long)(t0 + t) * C + c0 + 128 * j] = v;
+      }
+    }
   }
 }
 }  // namespace b200
@@ -369,11 +411,20 @@ B200_API int b200_lowrank_decay(const float* x, long long ldx, const float* w2, 
   using namespace b200;
   if (tokens <= 0) return 0;
   if (C <= 0 || rank <= 0 || tokens > 65535 * kLrTok) return B200_ERR_BAD_SHAPE;
-  const size_t smem = (size_t)kLrTok * rank * 4;
+  int groups = tokens >= 2048 ? 4 : 1;
+  while (groups > 1 && (size_t)groups * kLrTok * rank * 4 > 48 * 1024) groups /= 2;
+  const size_t smem = (size_t)groups * kLrTok * rank * 4;
   if (smem > 48 * 1024) return B200_ERR_TOO_LARGE;
-  dim3 grid((C + 127) / 128, (tokens + kLrTok - 1) / kLrTok);
-  if (fast) lowrank_decay_kernel<true><<<grid, 128, smem, (cudaStream_t)stream>>>(x, ldx, w2, bias, out, tokens, C, rank, inv_tau);
-  else lowrank_decay_kernel<false><<<grid, 128, smem, (cudaStream_t)stream>>>(x, ldx, w2, bias, out, tokens, C, rank, inv_tau);
+  const bool r16 = rank == 16 && !(reinterpret_cast<uintptr_t>(w2) & 15);
+  const int cpt = tokens >= 512 ? (r16 ? 2 : 4) : 1;
+  dim3 grid((C + 128 * cpt - 1) / (128 * cpt), (tokens + kLrTok * groups - 1) / (kLrTok * groups));
+#define LR(FF, CC, RR)                                                                                                         \
+  lowrank_decay_kernel<FF, CC, RR><<<grid, 128, smem, (cudaStream_t)stream>>>(x, ldx, w2, bias, out, tokens, C, rank, inv_tau, groups)
+#define LR_F(FF)                                                                                                               \
+  do { if (cpt == 2) LR(FF, 2, 16); else if (cpt == 4) LR(FF, 4, 0); else if (r16) LR(FF, 1, 16); else LR(FF, 1, 0); } while (0)
+  if (fast) LR_F(true); else LR_F(false);
+#undef LR_F
+#undef LR
   B200_LAUNCH_CHECK();
   return 0;
 }

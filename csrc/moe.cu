@@ -216,11 +216,13 @@ moe_dispatch_kernel(const long long* __restrict__ top_i, long long* __restrict__
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   for (int e = tid; e < E; e += blockDim.x) cnt[e] = 0;
   __syncthreads();
-  for (int r = tid; r < R; r += blockDim.x) {
-    const long long e = top_i[r];
+  for (int r0 = 0; r0 < R; r0 += blockDim.x) {                      // one atomic per expert that occurs in a warp's 32 ids
+    const int r = r0 + tid;
+    const long long e = r < R ? top_i[r] : -1;
     const bool ok = e >= 0 && e < E;
-    ids[r] = ok ? (unsigned short)e : (unsigned short)0xffff;
-    if (ok) atomicAdd(&cnt[(int)e], 1);
+    if (r < R) ids[r] = ok ? (unsigned short)e : (unsigned short)0xffff;
+    const unsigned same = __match_any_sync(0xffffffffu, ok ? (int)e : -1);
+    if (ok && lane == __ffs(same) - 1) atomicAdd(&cnt[(int)e], __popc(same));
   }
   __syncthreads();
   if (tid == 0) {

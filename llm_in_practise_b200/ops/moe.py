@@ -105,13 +105,14 @@ def _grouped_ref(xs, tile_map, w, b, tile):
 
 
 def _grouped_gemm(a: torch.Tensor, w: torch.Tensor, tile_map: torch.Tensor, bias: Optional[torch.Tensor], b_mn: bool,
-                  tile: int) -> torch.Tensor:
-    """a [NT*tile, Ka]; w [E, N, K]; forward (b_mn False): out[t] = a[t] w[e]^T (+ bias[e]); dgrad (b_mn True): a[t] w[e]."""
+                  tile: int, zero: bool = True) -> torch.Tensor:
+    """``zero`` False: unused tiles of the result are left as they are (inference never reads them).
+    a [NT*tile, Ka]; w [E, N, K]; forward (b_mn False): out[t] = a[t] w[e]^T (+ bias[e]); dgrad (b_mn True): a[t] w[e]."""
     nt = tile_map.numel()
     E, N, K = w.shape
     n_out = K if b_mn else N
     a3 = a.view(nt, tile, a.shape[-1])
-    out = torch.zeros(nt, tile, n_out, dtype=a.dtype, device=a.device)
+    out = (torch.zeros if zero else torch.empty)(nt, tile, n_out, dtype=a.dtype, device=a.device)
     args = nv.GemmArgs()
     args.A, args.B, args.D = a3.data_ptr(), w.data_ptr(), out.data_ptr()
     args.bias = 0 if bias is None else bias.data_ptr()
@@ -166,6 +167,8 @@ def grouped_linear(xs: torch.Tensor, w: torch.Tensor, b: Optional[torch.Tensor],
     """xs [d.rows, K] (expert-sorted, tile-padded) -> [d.rows, N]: row tile t uses w[tile_map[t]] / b[tile_map[t]]."""
     if (nv.use_native(xs) and xs.dtype in (torch.bfloat16, torch.float16) and w.dtype == xs.dtype and tile == TILE
             and xs.shape[-1] % 8 == 0 and w.shape[1] % 8 == 0 and xs.is_contiguous() and w.is_contiguous()):
+        if not torch.is_grad_enabled():
+            return _grouped_gemm(xs, w, d.tile_map, b, False, tile, zero=False)
         return _GroupedLinearFn.apply(xs, w, b, d, tile)
     return _grouped_ref(xs, d.tile_map, w, b, tile)
 
