@@ -22,8 +22,9 @@ Layer i (tensors ``l<i>.*``), m = ``residual_mult``:
 
 A layer with ``weights_of: j`` runs layer j's tensors again with pages and state of its own. The output is
 ``embed @ (RMS(x) * g)`` (the embedding table without its scale). What is fp32 whatever the model dtype: the stream, every
-norm, attention scores and softmax, the router, the recurrent states and everything between the projections (short
-convolutions included) and the scans: decays, step sizes, read-outs and their norms.
+norm, attention scores and softmax, the router, the recurrent states and tails, decays, step sizes, the scans and their
+read-outs. Projections, the rows that leave a short convolution, B and C are in the model dtype where they do not feed the
+matrix memory (whose projections are written in fp32).
 
 Keys and values live in the paged cache (``kv_layout``), convolution tails and recurrent states in its per-sequence state rows
 (``state_layout``). ``inference/ragged.RaggedGenerator`` and ``serve/engine.LLMEngine`` drive ``forward_ragged``.
