@@ -27,8 +27,8 @@ NATIVE_SOURCES = {
                 "linear_scan"],
     "Kudonex": ["gemm_tcgen05", "gemv", "gemm_simt", "norm", "elementwise", "paged_attn", "moe", "linear_scan", "talking_attn",
                 "talking_attn_mma"],
-    "Lorenex": ["gemm_tcgen05", "gemv", "gemm_simt", "norm", "elementwise", "moe", "linear_scan", "selective_scan", "multimap_attn",
-                "multimap_attn_mma"],
+    "Lorenex": ["gemm_tcgen05", "gemv", "gemm_simt", "norm", "elementwise", "moe", "linear_scan", "channel_scan", "selective_scan",
+                "multimap_attn", "multimap_attn_mma"],
 }
 BLOCK = 64
 MAX_LIVE = 4

@@ -680,3 +680,23 @@ def test_checkpoint_names_round_trip_and_bad_configs(tmp_path):
         breakage(bad)
         with pytest.raises(ValueError):
             LorenexConfig.from_dict(bad)
+
+
+def test_replay_builds_every_kernel_source_the_model_calls():
+    """A fresh checkout compiles only the sources listed for the design: each entry point the model's ops call is in one."""
+    import inspect
+    import re
+    from llm_in_practise_b200 import _build
+    from llm_in_practise_b200.ops import elementwise, gemm, linear_scan, moe, multimap_attention, norm
+    from llm_in_practise_b200.recipes.trace import NATIVE_SOURCES
+    have = set()
+    for stem in NATIVE_SOURCES["Lorenex"]:
+        have |= set(re.findall(r"B200_API int (b200_\w+)\(", (_build.CSRC / f"{stem}.cu").read_text()))
+    called = set()
+    for fn in (elementwise.embedding_pos, elementwise.clamped_glu, gemm.gemm, gemm.gemv16, gemm.linear_exact, linear_scan.linear_scan,
+               linear_scan.lowrank_decay, linear_scan.scan_readout, linear_scan.selective_scan, linear_scan.short_conv, linear_scan._conv_tail,
+               moe.route_grouped, moe.dispatch, moe.gather_rows, moe._grouped_gemm, moe.moe_combine, multimap_attention.conv_qknorm_store,
+               multimap_attention.multimap_attention, norm.poly_norm, norm.sandwich_norm):
+        called |= set(re.findall(r"\b(b200_\w+)\b", inspect.getsource(fn)))
+    called -= {"b200_gemm_args"}
+    assert len(called) > 15 and called <= have, sorted(called - have)
