@@ -199,8 +199,10 @@ def kernel_rows(size, dev, steps, warmup, root):
     qs, ks, aa, bb = rnd(T, SG * SD), rnd(T, SG * SD), rnd(T, SH * SD), rnd(T, SH)
     dtb, alog = torch.zeros(SH * SD, device=dev), torch.zeros(SH, device=dev)
     ms_l = t(lambda: delta_gates(qs, ks, aa, bb, dtb, alog, SG, SH, SD, 1.0), steps, warmup)
-    rows.append((f"per-channel decays from a rank-{rank} input, {SH * SD} channels", ms_k, frac_bw(T * SH * SD * 4, ms_k),
-                 "Duratar: unit q / k, decays, beta", ms_l, frac_bw(T * (2 * SG * SD + SH * SD + SH) * 8, ms_l), "HBM"))
+    roof = max(frac_bw(T * SH * SD * 4, ms_k), 3 * T * SH * SD / (ms_k * 1e-3) / 1e12 / EXP_RATE)     # two exponentials, one logarithm
+    rows.append((f"per-channel decays from a rank-{rank} input, {SH * SD} channels", ms_k, roof,
+                 "Duratar: unit q / k, decays, beta", ms_l, frac_bw(T * (2 * SG * SD + SH * SD + SH) * 8, ms_l),
+                 "slower of HBM and special-function rate; Duratar: HBM"))
     # --- matrix memory: prompt and decode batch
     g = lowrank_decay(a1, a2, ab, 16.0, fast=True)
     q16, k16, vs = rnd(T, SH * SD) * SD ** -0.5, rnd(T, SH * SD) * SD ** -0.5, rnd(T, SH * SDv)
