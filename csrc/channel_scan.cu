@@ -1,9 +1,12 @@
 // Gated linear attention with a decay per key channel, over the runs of a ragged serving step (see linear_scan.cu for runs,
 // state rows and the other scan modes). All arithmetic is fp32.
 //
-//   b200_lowrank_decay   a[t, c] = sigmoid(sum_r w2[c, r] x[t, r] + bias[c])^(1 / tau), formed as exp(log sigmoid(.) / tau)
+//   b200_lowrank_decay   a[t, c] = sigmoid(sum_r w2[c, r] x[t, r] + bias[c])^(1 / tau), formed as exp(log sigmoid(.) / tau), or
+//                        exp(-exp(sum_r w2[c, r] tanh(x[t, r]) + bias[c]))
 //   b200_channel_scan    per head, state S [D, Dv] (fp32, in `state` [rows, H, D, Dv]):
-//                            S <- diag(g_t) S + k_t v_t^T ;   o_t = S^T q_t
+//                            S <- diag(g_t) S + k_t v_t^T ;   o_t = S^T q_t                      (u NULL)
+//                            o_t = (S + diag(u) k_t v_t^T)^T q_t ;   S <- diag(g_t) S + k_t v_t^T  (u [H, D]: a bonus for the
+//                            current token, which the read-out sees before the state decays)
 //
 // A run is walked token by token, but the recurrence is linear, so a long run need not be walked by one CTA: it is cut into
 // tiles (64 tokens), and
@@ -33,7 +36,7 @@ __device__ __forceinline__ void cs_commit() { asm volatile("cp.async.commit_grou
 template <int N> __device__ __forceinline__ void cs_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
 struct ChannelScanArgs {
-  const float *q, *k, *v, *g;
+  const float *q, *k, *v, *g, *u;
   long long ldq, ldk, ldv, ldg;
   float* state;                                          // [rows, H, D, Dv]
   float* part;                                           // [tiles, H, D, Dv]: local, then incoming states
@@ -45,7 +48,7 @@ struct ChannelScanArgs {
 };
 
 // PASS 0: blockIdx.x is a run; 1, 2: a tile
-template <int PASS, int LPC>
+template <int PASS, int LPC, bool BONUS>
 __global__ void __launch_bounds__(128)
 channel_scan_kernel(const ChannelScanArgs a) {
   extern __shared__ __align__(16) float sm[];
@@ -121,6 +124,15 @@ channel_scan_kernel(const ChannelScanArgs a) {
 #pragma unroll
   for (int i = 0; i < R / 2; ++i) P2[i] = make_float2(1.f, 1.f);
 
+  float2 u2[R / 2];
+  if (BONUS && PASS != 1) {
+#pragma unroll
+    for (int i = 0; i < R / 2; ++i) {
+      u2[i].x = row0 + 2 * i < D ? a.u[h * D + row0 + 2 * i] : 0.f;
+      u2[i].y = row0 + 2 * i + 1 < D ? a.u[h * D + row0 + 2 * i + 1] : 0.f;
+    }
+  }
+
   auto stage = [&](int b, int c0) {
     const int cn = min(CH, n - c0);
     for (int tt = warp; tt < cn; tt += nw) {
@@ -185,16 +197,25 @@ channel_scan_kernel(const ChannelScanArgs a) {
       const float4 vv = *reinterpret_cast<const float4*>(vs + tt * ncol);
       const float vc[CPT] = {vv.x, vv.y, vv.z, vv.w};
       float o[CPT];
+      float bonus = 0.f;                                 // this lane's part of q . diag(u) k, the weight of the token's own value
+      if (BONUS && PASS != 1) {
+        float2 ba = make_float2(0.f, 0.f);
+#pragma unroll
+        for (int i = 0; i < R / 2; ++i) ba = __ffma2_rn(__fmul2_rn(u2[i], k2[i]), q2[i], ba);
+        bonus = ba.x + ba.y;
+      }
 #pragma unroll
       for (int c = 0; c < CPT; ++c) {
         const float2 v2 = make_float2(vc[c], vc[c]);
         float2 oa = make_float2(0.f, 0.f);
 #pragma unroll
         for (int i = 0; i < R / 2; ++i) {
+          if (BONUS && PASS != 1) oa = __ffma2_rn(S2[c][i], q2[i], oa);
           S2[c][i] = __ffma2_rn(g2[i], S2[c][i], __fmul2_rn(k2[i], v2));
-          if (PASS != 1) oa = __ffma2_rn(S2[c][i], q2[i], oa);
+          if (!BONUS && PASS != 1) oa = __ffma2_rn(S2[c][i], q2[i], oa);
         }
         o[c] = oa.x + oa.y;
+        if (BONUS && PASS != 1) o[c] = fmaf(bonus, vc[c], o[c]);
       }
       if (PASS == 1) {
         if (owns_dec) {
@@ -311,7 +332,8 @@ channel_scan_carry_kernel(float* __restrict__ part, const float* __restrict__ pd
 // add up where the rounding of 1 + expm1 does not.
 constexpr int kLrTok = 8;
 // CPT channels per thread share the reads of x. RK: the rank at compile time, weights then stay in registers (0: any rank)
-template <bool FAST, int CPT, int RK>
+// EXPO: the inputs pass tanh as they are staged, and the decay is exp(-exp(z)).
+template <bool FAST, int CPT, int RK, bool EXPO>
 __global__ void __launch_bounds__(128)
 lowrank_decay_kernel(const float* __restrict__ x, long long ldx, const float* __restrict__ w2, const float* __restrict__ bias,
                      float* __restrict__ out, int tokens, int C, int rank, float inv_tau, int groups) {
@@ -319,7 +341,8 @@ lowrank_decay_kernel(const float* __restrict__ x, long long ldx, const float* __
   const int tb = blockIdx.y * kLrTok * groups;
   for (int i = threadIdx.x; i < groups * kLrTok * rank; i += blockDim.x) {
     const int t = i / rank;
-    xall[i] = tb + t < tokens ? x[(long long)(tb + t) * ldx + i % rank] : 0.f;
+    const float xv = tb + t < tokens ? x[(long long)(tb + t) * ldx + i % rank] : 0.f;
+    xall[i] = EXPO ? tanhf(xv) : xv;
   }
   __syncthreads();
   const int c0 = blockIdx.x * 128 * CPT + threadIdx.x;   // this thread's channels are 128 apart
@@ -392,7 +415,10 @@ lowrank_decay_kernel(const float* __restrict__ x, long long ldx, const float* __
       for (int j = 0; j < CPT; ++j) {
         const float z = acc[t][j];
         float v;
-        if (FAST) {
+        if (EXPO) {
+          const float y = -expf(z);
+          v = FAST ? ex2_approx(y * 1.4426950408889634f) : (y > -0.5f ? 1.f + expm1f(y) : expf(y));
+        } else if (FAST) {
           const float z2 = z * 1.4426950408889634f;
           v = ex2_approx((fminf(z2, 0.f) - __log2f(1.f + ex2_approx(-fabsf(z2)))) * inv_tau);
         } else {
@@ -406,8 +432,9 @@ lowrank_decay_kernel(const float* __restrict__ x, long long ldx, const float* __
 }
 }  // namespace b200
 
-B200_API int b200_lowrank_decay(const float* x, long long ldx, const float* w2, const float* bias, float* out, int tokens, int C,
-                                int rank, float inv_tau, int fast, void* stream) {
+// form 0: sigmoid(w2 x + bias)^inv_tau; 1: exp(-exp(w2 tanh(x) + bias))
+B200_API int b200_lowrank_decay_ex(const float* x, long long ldx, const float* w2, const float* bias, float* out, int tokens, int C,
+                                   int rank, float inv_tau, int form, int fast, void* stream) {
   using namespace b200;
   if (tokens <= 0) return 0;
   if (C <= 0 || rank <= 0 || tokens > 65535 * kLrTok) return B200_ERR_BAD_SHAPE;
@@ -419,7 +446,10 @@ B200_API int b200_lowrank_decay(const float* x, long long ldx, const float* w2, 
   const int cpt = tokens >= 512 ? (r16 ? 2 : 4) : 1;
   dim3 grid((C + 128 * cpt - 1) / (128 * cpt), (tokens + kLrTok * groups - 1) / (kLrTok * groups));
 #define LR(FF, CC, RR)                                                                                                         \
-  lowrank_decay_kernel<FF, CC, RR><<<grid, 128, smem, (cudaStream_t)stream>>>(x, ldx, w2, bias, out, tokens, C, rank, inv_tau, groups)
+  do {                                                                                                                         \
+    if (form == 1) lowrank_decay_kernel<FF, CC, RR, true><<<grid, 128, smem, (cudaStream_t)stream>>>(x, ldx, w2, bias, out, tokens, C, rank, inv_tau, groups); \
+    else lowrank_decay_kernel<FF, CC, RR, false><<<grid, 128, smem, (cudaStream_t)stream>>>(x, ldx, w2, bias, out, tokens, C, rank, inv_tau, groups); \
+  } while (0)
 #define LR_F(FF)                                                                                                               \
   do { if (cpt == 2) LR(FF, 2, 16); else if (cpt == 4) LR(FF, 4, 0); else if (r16) LR(FF, 1, 16); else LR(FF, 1, 0); } while (0)
   if (fast) LR_F(true); else LR_F(false);
@@ -429,8 +459,13 @@ B200_API int b200_lowrank_decay(const float* x, long long ldx, const float* w2, 
   return 0;
 }
 
+B200_API int b200_lowrank_decay(const float* x, long long ldx, const float* w2, const float* bias, float* out, int tokens, int C,
+                                int rank, float inv_tau, int fast, void* stream) {
+  return b200_lowrank_decay_ex(x, ldx, w2, bias, out, tokens, C, rank, inv_tau, 0, fast, stream);
+}
+
 B200_API int b200_channel_scan(const float* q, long long ldq, const float* k, long long ldk, const float* v, long long ldv,
-                               const float* g, long long ldg, float* state, float* part, float* pdec, const int* runs, int n_runs,
+                               const float* g, long long ldg, const float* u, float* state, float* part, float* pdec, const int* runs, int n_runs,
                                const int* tiles, int n_tiles, const int* tile_of, const int* run_tiles, int chunk, const int* pos, const int* slot, float* o,
                                int H, int G, int D, int Dv, void* stream) {
   using namespace b200;
@@ -450,16 +485,17 @@ B200_API int b200_channel_scan(const float* q, long long ldq, const float* k, lo
   while (CH > 1 && bytes(CH) > 100 * 1024) CH /= 2;
   auto al = [](const void* p_, long long ld) { return !(reinterpret_cast<uintptr_t>(p_) & 15) && ld % 4 == 0; };
   ChannelScanArgs a;
-  a.q = q; a.k = k; a.v = v; a.g = g; a.ldq = ldq; a.ldk = ldk; a.ldv = ldv; a.ldg = ldg;
+  a.q = q; a.k = k; a.v = v; a.g = g; a.u = u; a.ldq = ldq; a.ldk = ldk; a.ldv = ldv; a.ldg = ldg;
   a.state = state; a.part = part; a.pdec = pdec; a.runs = runs; a.pos = pos; a.slot = slot; a.tiles = tiles; a.tile_of = tile_of;
   a.o = o; a.H = H; a.G = G; a.D = D; a.Dv = Dv; a.chunk = CH;
   a.vec = D % 4 == 0 && al(q, ldq) && al(k, ldk) && al(g, ldg);
   a.vecv = Dv % 4 == 0 && al(v, ldv) && al(state, 4) && al(o, 4) && (!part || al(part, 4));
   cudaStream_t st = (cudaStream_t)stream;
   const size_t smem = bytes(CH);
-#define CS(PASS, LL, NB)                                                                                                   \
+#define CS(PASS, LL, NB) do { if (u) CS_B(PASS, LL, NB, true); else CS_B(PASS, LL, NB, false); } while (0)
+#define CS_B(PASS, LL, NB, BB)                                                                                             \
   do {                                                                                                                     \
-    auto kern = channel_scan_kernel<PASS, LL>;                                                                             \
+    auto kern = channel_scan_kernel<PASS, LL, (PASS != 1 && BB)>;                                                                             \
     if (smem > 48 * 1024) B200_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));  \
     kern<<<dim3(NB, H, zb), nw * 32, smem, st>>>(a);                                                                       \
   } while (0)
@@ -480,6 +516,7 @@ B200_API int b200_channel_scan(const float* q, long long ldq, const float* k, lo
     CS_L(2, n_tiles);
   }
 #undef CS_L
+#undef CS_B
 #undef CS
   B200_LAUNCH_CHECK();
   return 0;

@@ -469,15 +469,15 @@ B200_API int b200_embedding_fwd(const long long* ids, const void* table, const v
 }
 namespace b200 {
 // out[t, c] = table[ids[t], c] * scale + pos_table[pos[t], c]: embedding rows entering an fp32 stream with an additive
-// position table (fp32, built on the host) indexed by every token's own position
+// position table (fp32, built on the host) indexed by every token's own position, or without one (NULL)
 template <typename T>
 __global__ void embedding_pos_kernel(const long long* __restrict__ ids, const T* __restrict__ table, float scale,
                                      const int* __restrict__ pos, const float* __restrict__ pos_table, float* __restrict__ out,
                                      int dim) {
   const long long t = blockIdx.x;
   const T* src = table + ids[t] * dim;
-  const float* ps = pos_table + (long long)pos[t] * dim;
-  for (int i = threadIdx.x; i < dim; i += blockDim.x) out[t * dim + i] = fmaf(to_f32<T>(src[i]), scale, ps[i]);
+  const float* ps = pos_table ? pos_table + (long long)pos[t] * dim : nullptr;
+  for (int i = threadIdx.x; i < dim; i += blockDim.x) out[t * dim + i] = fmaf(to_f32<T>(src[i]), scale, ps ? ps[i] : 0.f);
 }
 }  // namespace b200
 

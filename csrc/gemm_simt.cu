@@ -1,4 +1,4 @@
-// D[M, N] = A[M, K] B[N, K]^T in true fp32 (FFMA, sequential-k accumulation per output): the exact-precision path for
+// D[M, N] = A[M, K] B[N, K]^T (+ bias[N]) in true fp32 (FFMA, sequential-k accumulation per output): the exact-precision path for
 // fp32 inference, where the tensor-core route would round the operands to TF32. 64 x 64 tiles, 16-deep k steps, 4 x 4
 // outputs per thread; any M, N, K and any row strides.
 #include "common.cuh"
@@ -8,8 +8,8 @@ namespace b200 {
 constexpr int kSB = 64, kSK = 16;
 
 __global__ void __launch_bounds__(256)
-gemm_f32_kernel(const float* __restrict__ A, const float* __restrict__ B, float* __restrict__ D, int M, int N, int K,
-                long long lda, long long ldb, long long ldd) {
+gemm_f32_kernel(const float* __restrict__ A, const float* __restrict__ B, const float* __restrict__ bias, float* __restrict__ D,
+                int M, int N, int K, long long lda, long long ldb, long long ldd) {
   __shared__ float As[kSK][kSB + 4];
   __shared__ float Bs[kSK][kSB + 4];
   const int tx = threadIdx.x % 16, ty = threadIdx.x / 16;
@@ -38,17 +38,22 @@ gemm_f32_kernel(const float* __restrict__ A, const float* __restrict__ B, float*
   for (int i = 0; i < 4; ++i)
     for (int j = 0; j < 4; ++j) {
       const int gm = m0 + ty * 4 + i, gn = n0 + tx * 4 + j;
-      if (gm < M && gn < N) D[(long long)gm * ldd + gn] = acc[i][j];
+      if (gm < M && gn < N) D[(long long)gm * ldd + gn] = acc[i][j] + (bias ? bias[gn] : 0.f);
     }
 }
 }  // namespace b200
 
-B200_API int b200_gemm_f32_exact(const float* A, const float* B, float* D, int M, int N, int K, long long lda, long long ldb,
-                                 long long ldd, void* stream) {
+B200_API int b200_gemm_f32_exact_bias(const float* A, const float* B, const float* bias, float* D, int M, int N, int K, long long lda,
+                                      long long ldb, long long ldd, void* stream) {
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0) return B200_ERR_BAD_SHAPE;
   dim3 grid((N + b200::kSB - 1) / b200::kSB, (M + b200::kSB - 1) / b200::kSB);
-  b200::gemm_f32_kernel<<<grid, 256, 0, (cudaStream_t)stream>>>(A, B, D, M, N, K, lda, ldb, ldd);
+  b200::gemm_f32_kernel<<<grid, 256, 0, (cudaStream_t)stream>>>(A, B, bias, D, M, N, K, lda, ldb, ldd);
   B200_LAUNCH_CHECK();
   return 0;
+}
+
+B200_API int b200_gemm_f32_exact(const float* A, const float* B, float* D, int M, int N, int K, long long lda, long long ldb,
+                                 long long ldd, void* stream) {
+  return b200_gemm_f32_exact_bias(A, B, nullptr, D, M, N, K, lda, ldb, ldd, stream);
 }

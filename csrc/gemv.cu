@@ -84,6 +84,7 @@ struct GemvParams {
   int gshift;             // log2(group) when it is a power of two, else -1
   float lin_a, lin_off;   // LIN: lut[code] = lin_a * (code - lin_off), lin_off an integer
   long long N, x_rs, w_rs, y_rs;
+  long long x_bs, w_bs, y_bs;   // dense only: problem blockIdx.y starts this many elements further
   // ---- fused tail (fuse != 0): the product never goes to a y tensor of its own. Every CTA writes its 16-column tiles into
   // a staging buffer (fuse 1: local; fuse 2: this rank's half of a symmetric buffer, tensor-parallel row-parallel layer),
   // a ticket barrier closes the GEMV, (fuse 2) the epoch is published to the peers and theirs awaited, and CTA m then
@@ -134,6 +135,7 @@ gemv_mma_kernel(const GemvParams p) {
   const int g = lane >> 2, t = lane & 3;
   const int K = p.K, M = p.M;
   const long long N = p.N;
+  const uint16_t* px = p.x + blockIdx.y * p.x_bs;
   // activations -> shared memory once per CTA (the host sized the allocation; 16-byte padded rows)
   const bool xsm = (long long)M * (K + 8) * 2 <= 73728;
   uint16_t* xs = reinterpret_cast<uint16_t*>(table + ((W4 && !LIN) ? 256 * 32 : 0));
@@ -141,12 +143,13 @@ gemv_mma_kernel(const GemvParams p) {
     const int vpr = K / 8;
     for (int i = threadIdx.x; i < M * vpr; i += 256) {
       const int r = i / vpr, cvec = i - r * vpr;
-      *reinterpret_cast<uint4*>(xs + (long long)r * (K + 8) + cvec * 8) = __ldg(reinterpret_cast<const uint4*>(p.x + (long long)r * p.x_rs) + cvec);
+      *reinterpret_cast<uint4*>(xs + (long long)r * (K + 8) + cvec * 8) = __ldg(reinterpret_cast<const uint4*>(px + (long long)r * p.x_rs) + cvec);
     }
     __syncthreads();
   }
   uint32_t epoch = 0;
   void* ybase = p.y;
+  if (blockIdx.y) ybase = p.out_f32 ? (void*)(reinterpret_cast<float*>(p.y) + blockIdx.y * p.y_bs) : (void*)(reinterpret_cast<uint16_t*>(p.y) + blockIdx.y * p.y_bs);
   long long y_rs = p.y_rs;
   if (p.fuse) {
     epoch = *((volatile unsigned int*)p.state) + 1u;
@@ -263,7 +266,7 @@ gemv_mma_kernel(const GemvParams p) {
           }
         }
       } else {
-        const uint16_t* wd = reinterpret_cast<const uint16_t*>(p.w);
+        const uint16_t* wd = reinterpret_cast<const uint16_t*>(p.w) + blockIdx.y * p.w_bs;
         const uint4* pa = reinterpret_cast<const uint4*>(wd + rA * p.w_rs + k);
         const uint4* pb = reinterpret_cast<const uint4*>(wd + rB * p.w_rs + k);
 #pragma unroll
@@ -279,7 +282,7 @@ gemv_mma_kernel(const GemvParams p) {
         uint32_t xw[16];
         if (tok < M) {
           const uint4* xp = xsm ? reinterpret_cast<const uint4*>(xs + (long long)tok * (K + 8) + k)
-                                : reinterpret_cast<const uint4*>(p.x + (long long)tok * p.x_rs + k);
+                                : reinterpret_cast<const uint4*>(px + (long long)tok * p.x_rs + k);
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
             const uint4 v = xsm ? xp[i] : __ldg(xp + i);
@@ -465,7 +468,7 @@ gemv_mma_kernel(const GemvParams p) {
 }
 
 template <bool BF16, bool W4, int TG, int MINB, bool LIN = false, bool POST = false>
-static cudaError_t launch_gemv_one(const GemvParams& p_in, cudaStream_t st) {
+static cudaError_t launch_gemv_one(const GemvParams& p_in, cudaStream_t st, int batch = 1) {
   GemvParams p = p_in;
   p.gshift = (p.group > 0 && (p.group & (p.group - 1)) == 0) ? __builtin_ctz(p.group) : -1;
   // persistent over 16-row tiles: one resident wave (occupancy x SMs), never more CTAs than tiles
@@ -483,8 +486,9 @@ static cudaError_t launch_gemv_one(const GemvParams& p_in, cudaStream_t st) {
     if (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&occ, gemv_mma_kernel<BF16, W4, TG, MINB, LIN, POST>, 256, smem) != cudaSuccess || occ < 1) occ = 1;
   }
   const long long tiles = (p.N + 15) / 16;
-  const unsigned grid = (unsigned)(tiles < (long long)kNumSMs * occ ? tiles : (long long)kNumSMs * occ);
-  return launch_pdl(gemv_mma_kernel<BF16, W4, TG, MINB, LIN, POST>, grid, 256, smem, st, p);
+  const long long wave = ((long long)kNumSMs * occ + batch - 1) / batch;
+  const unsigned grid = (unsigned)(tiles < wave ? tiles : wave);
+  return launch_pdl(gemv_mma_kernel<BF16, W4, TG, MINB, LIN, POST>, dim3(grid, batch), 256, smem, st, p);
 }
 
 template <bool BF16>
@@ -509,15 +513,15 @@ static int launch_gemv_lin(const GemvParams& p, cudaStream_t st) {
 }
 
 template <bool BF16, bool W4>
-static int launch_gemv(const GemvParams& p, cudaStream_t st) {
+static int launch_gemv(const GemvParams& p, cudaStream_t st, int batch = 1) {
   // dense weights: registers cap the occupancy (96 -> 2 CTAs per SM); forcing 3 trades a few spills for 50 % more loads in
   // flight, which is what a weight-streaming kernel is short of (B200_GEMV_MINB=2|3|4 to compare)
   static const int minb = [] { const char* e = getenv("B200_GEMV_MINB"); return e ? atoi(e) : 0; }();
   cudaError_t e;
 #define B200_GV(TGv)                                                                     \
-  (W4 || minb == 0 || minb == 2 ? launch_gemv_one<BF16, W4, TGv, W4 ? 1 : 2>(p, st)        \
-   : minb == 3                  ? launch_gemv_one<BF16, W4, TGv, W4 ? 1 : 3>(p, st)        \
-                                : launch_gemv_one<BF16, W4, TGv, W4 ? 1 : 4>(p, st))
+  (W4 || minb == 0 || minb == 2 ? launch_gemv_one<BF16, W4, TGv, W4 ? 1 : 2>(p, st, batch) \
+   : minb == 3                  ? launch_gemv_one<BF16, W4, TGv, W4 ? 1 : 3>(p, st, batch) \
+                                : launch_gemv_one<BF16, W4, TGv, W4 ? 1 : 4>(p, st, batch))
   if (p.M <= 8) e = B200_GV(1);
   else if (p.M <= 16) e = B200_GV(2);
   else if (p.M <= 32) e = B200_GV(4);
@@ -529,16 +533,23 @@ static int launch_gemv(const GemvParams& p, cudaStream_t st) {
 }  // namespace b200
 using namespace b200;
 
-B200_API int b200_gemv16(const void* x, const void* w, const void* bias, void* y, int M, long long N, int K, long long x_rs,
-                         long long w_rs, long long y_rs, int dtype, int out_f32, void* stream) {
-  if (M < 1 || M > 64 || K % 128 || x_rs % 8 || w_rs % 8) return B200_ERR_BAD_SHAPE;
+B200_API int b200_gemv16_batched(const void* x, const void* w, const void* bias, void* y, int M, long long N, int K, long long x_rs,
+                                 long long w_rs, long long y_rs, int batch, long long x_bs, long long w_bs, long long y_bs, int dtype,
+                                 int out_f32, void* stream) {
+  if (M < 1 || M > 64 || K % 128 || x_rs % 8 || w_rs % 8 || x_bs % 8 || w_bs % 8 || batch < 1 || batch > 65535) return B200_ERR_BAD_SHAPE;
   if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) return B200_ERR_BAD_ALIGN;
   GemvParams p = {};
   p.x = (const uint16_t*)x; p.w = w; p.bias = bias; p.y = y;
   p.M = M; p.K = K; p.N = N; p.x_rs = x_rs; p.w_rs = w_rs; p.y_rs = y_rs; p.out_f32 = out_f32; p.group = 128;
-  if (dtype == B200_DT_BF16) return launch_gemv<true, false>(p, (cudaStream_t)stream);
-  if (dtype == B200_DT_FP16) return launch_gemv<false, false>(p, (cudaStream_t)stream);
+  p.x_bs = x_bs; p.w_bs = w_bs; p.y_bs = y_bs;
+  if (dtype == B200_DT_BF16) return launch_gemv<true, false>(p, (cudaStream_t)stream, batch);
+  if (dtype == B200_DT_FP16) return launch_gemv<false, false>(p, (cudaStream_t)stream, batch);
   return B200_ERR_UNSUPPORTED;
+}
+
+B200_API int b200_gemv16(const void* x, const void* w, const void* bias, void* y, int M, long long N, int K, long long x_rs,
+                         long long w_rs, long long y_rs, int dtype, int out_f32, void* stream) {
+  return b200_gemv16_batched(x, w, bias, y, M, N, K, x_rs, w_rs, y_rs, 1, 0, 0, 0, dtype, out_f32, stream);
 }
 
 B200_API int b200_w4_gemv_batched(const void* x, const uint8_t* packed, const float* scale, const float* zs, const float* lut,

@@ -12,12 +12,14 @@
 //                          scan without a convolution, done once instead of by every CTA that reads them).
 //   b200_short_conv_tail   advances that tail over the step's runs (launched after the convolution has read the old one); for
 //                          a decode batch the convolution does it itself. `in_bias`: a bias that belongs to the inputs.
-//   b200_delta_gates       q, k -> unit vectors per head (q also times `qscale`); a -> exp(-exp(A_log[h]) softplus(a + bias));
-//                          b -> sigmoid(b); in place, fp32.
+//   b200_delta_gates       q, k -> unit vectors per head (q also times `qscale`); a -> exp(-exp(A_log[h]) softplus(a + bias)),
+//                          one per key channel or one per head; b -> sigmoid(b); in place, fp32.
+//   b200_token_shift       several mixes of every token with the one before it, h + (h' - h) mu_s, h' carried like a tail.
 //   b200_linear_scan       per head, state S [D, Dv] (fp32, in `state` [rows, H, D, Dv]):
 //                            mode 0  S <- decay_h S + k v^T ;                                   o = S^T q
 //                            mode 1  S <- diag(g) S ; u = beta (v - S^T k) ; S <- S + k u^T ;   o = S^T q
 //                            mode 2  S <- a_t S + b_t k v^T  (a, b one number per token and head) ;   o = S^T q
+//                            mode 3  mode 1 with one decay per token and head
 //                          `ones` appends a column of ones to v (the state's last column is then the decayed sum of the
 //                          b_t k_t, and o's last column its product with q: the normaliser of an mLSTM read-out).
 //   b200_mlstm_gates       capped log gates of an mLSTM with their running maximum m (carried per sequence and head):
@@ -207,8 +209,8 @@ __global__ void short_conv_tail_kernel(const TX* __restrict__ x, long long ldx, 
 __global__ void __launch_bounds__(128)
 delta_gates_kernel(float* __restrict__ q, long long ldq, float* __restrict__ k, long long ldk, float* __restrict__ a,
                    long long lda, float* __restrict__ b, long long ldb, const float* __restrict__ dt_bias,
-                   const float* __restrict__ A_log, int G, int H, int D, float qscale, float unit_eps) {
-  const int t = blockIdx.x;
+                   const float* __restrict__ A_log, int G, int H, int D, int AD, float qscale, float unit_eps) {
+  const int t = blockIdx.x;                               // AD: decays per head (D, or 1)
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   for (int r = warp; r < 2 * G + H; r += nw) {
     if (r < 2 * G) {
@@ -220,10 +222,10 @@ delta_gates_kernel(float* __restrict__ q, long long ldq, float* __restrict__ k, 
       for (int d = lane; d < D; d += 32) x[d] *= sc;
     } else {
       const int h = r - 2 * G;
-      float* x = a + (long long)t * lda + (long long)h * D;
+      float* x = a + (long long)t * lda + (long long)h * AD;
       const float rate = expf(A_log[h]);
-      for (int d = lane; d < D; d += 32) {
-        const float z = x[d] + dt_bias[h * D + d];
+      for (int d = lane; d < AD; d += 32) {
+        const float z = x[d] + dt_bias[h * AD + d];
         const float sp = z > 20.f ? z : log1pf(expf(z));
         x[d] = expf(-rate * sp);
       }
@@ -232,6 +234,45 @@ delta_gates_kernel(float* __restrict__ q, long long ldq, float* __restrict__ k, 
   for (int h = threadIdx.x; h < H; h += blockDim.x) {
     float* x = b + (long long)t * ldb + h;
     *x = 1.f / (1.f + expf(-*x));
+  }
+}
+
+// out[s, t, c] = h[t, c] + (h' - h[t, c]) mu[s, c], h' the previous token's h: the row before inside a run, else `prev`
+// [rows, W] (zeros at position 0). step_tail: every token is a run of its own, so the thread that read prev also replaces it.
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+token_shift_kernel(const T* __restrict__ h, long long ldh, const float* __restrict__ mu, float* __restrict__ prev,
+                   const int* __restrict__ pos, const int* __restrict__ slot, T* __restrict__ out, int tokens, int W, int S,
+                   int step_tail) {
+  const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  const int WV = W / V;
+  if (idx >= (long long)tokens * WV) return;
+  const int t = (int)(idx / WV), c = (int)(idx % WV) * V;
+  const int p = pos[t], s = slot[t];
+  float x[V], y[V];
+  load_f32<V, T>(h + (long long)t * ldh + c, x);
+#pragma unroll
+  for (int e = 0; e < V; ++e) y[e] = 0.f;
+  float* pr = prev + (long long)s * W + c;
+  if (p > 0) {
+    if (!step_tail && t > 0 && slot[t - 1] == s && pos[t - 1] == p - 1) load_f32<V, T>(h + (long long)(t - 1) * ldh + c, y);
+    else load_f32<V, float>(pr, y);
+  }
+  if (step_tail) {
+#pragma unroll
+    for (int e = 0; e < V; ++e) pr[e] = x[e];
+  }
+#pragma unroll
+  for (int e = 0; e < V; ++e) y[e] -= x[e];
+  for (int i = 0; i < S; ++i) {
+    float m[V], r[V];
+    load_f32<V, float>(mu + (long long)i * W + c, m);
+#pragma unroll
+    for (int e = 0; e < V; ++e) r[e] = fmaf(y[e], m[e], x[e]);
+    T* dst = out + ((long long)i * tokens + t) * W + c;
+    if (V == 4 && sizeof(T) == 4) *reinterpret_cast<float4*>(dst) = *reinterpret_cast<const float4*>(r);
+    else if (V == 4) *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16x2(r[0], r[1 % V]), pack_bf16x2(r[V > 2 ? 2 : 0], r[V - 1]));
+    else dst[0] = from_f32<T>(r[0]);
   }
 }
 
@@ -256,7 +297,9 @@ linear_scan_kernel(const float* __restrict__ q, long long ldq, const float* __re
                    const float* __restrict__ beta, long long ldb, const float* __restrict__ decay, float* __restrict__ state,
                    const int* __restrict__ runs, const int* __restrict__ pos, const int* __restrict__ slot,
                    float* __restrict__ o, int H, int G, int D, int Dv, int act, int vec, int ones) {
-  // MODE 2 reads its two per-token numbers through the pointers of mode 1's per-channel decays: g = a [T, H], beta = b [T, H]
+  // MODE 2 reads its two per-token numbers through the pointers of mode 1's per-channel decays: g = a [T, H], beta = b [T, H];
+  // MODE 3 likewise its decay and beta
+  constexpr bool DELTA = MODE == 1 || MODE == 3;
   extern __shared__ __align__(16) float sm[];
   const int r_ = blockIdx.x, h = blockIdx.y;
   int first, n, p0, s;
@@ -282,7 +325,7 @@ linear_scan_kernel(const float* __restrict__ q, long long ldq, const float* __re
   auto GS = [&](int b) { return sm + b * per + 2 * kScanChunk * DP; };                         // MODE 1 only
   auto VS = [&](int b) { return sm + b * per + (MODE == 1 ? 3 : 2) * kScanChunk * DP; };       // [chunk][ncp]
   auto BS = [&](int b) { return VS(b) + kScanChunk * ncp; };                                   // [chunk]
-  auto AS = [&](int b) { return VS(b) + kScanChunk * ncp + kScanChunk; };                      // [chunk], MODE 2 only
+  auto AS = [&](int b) { return VS(b) + kScanChunk * ncp + kScanChunk; };                      // [chunk], MODE 2 and 3 only
   float* os = sm + 2 * per;                               // [chunk][ncol][LPC]: per-lane parts of the read-outs of a chunk
   // padding rows (D <= d < DP) never arrive by copy: k = q = 0 (and a finite g) keep their state at zero
   if (LPC * R > D) {
@@ -331,7 +374,7 @@ linear_scan_kernel(const float* __restrict__ q, long long ldq, const float* __re
         else VS(b)[tt * ncp + cc] = 1.f;
       }
       if (MODE >= 1 && lane == 0) cp_async4(BS(b) + tt, beta + tr * ldb + h);
-      if (MODE == 2 && lane == 1) cp_async4(AS(b) + tt, g + tr * ldg + h);
+      if (MODE >= 2 && lane == 1) cp_async4(AS(b) + tt, g + tr * ldg + h);
     }
   };
 
@@ -370,7 +413,7 @@ linear_scan_kernel(const float* __restrict__ q, long long ldq, const float* __re
       }
       const float vj = MODE == 2 ? vsp[tt * ncp] * bs[tt] : vsp[tt * ncp];
       float2 oa = make_float2(0.f, 0.f), ob = make_float2(0.f, 0.f);
-      if (MODE != 1) {
+      if (!DELTA) {
         const float dt_ = MODE == 2 ? as[tt] : dec;
         const float2 v2 = make_float2(vj, vj), dec2 = make_float2(dt_, dt_);
 #pragma unroll
@@ -384,7 +427,8 @@ linear_scan_kernel(const float* __restrict__ q, long long ldq, const float* __re
         float2 da = make_float2(0.f, 0.f), db = make_float2(0.f, 0.f);
 #pragma unroll
         for (int i = 0; i < R / 2; i += 2) {
-          const float4 g4 = *reinterpret_cast<const float4*>(gs + tt * DP + l * RP + 2 * i);
+          const float a_ = MODE == 3 ? as[tt] : 0.f;
+          const float4 g4 = MODE == 3 ? make_float4(a_, a_, a_, a_) : *reinterpret_cast<const float4*>(gs + tt * DP + l * RP + 2 * i);
           S2[i] = __fmul2_rn(S2[i], make_float2(g4.x, g4.y));
           S2[i + 1] = __fmul2_rn(S2[i + 1], make_float2(g4.z, g4.w));
           da = __ffma2_rn(S2[i], kr[i], da);
@@ -551,11 +595,11 @@ __global__ void ssm_gates_kernel(const float* __restrict__ dt, long long ld, con
 
 // One CTA per token; the row [N = H * Dv] lives in shared memory between the passes. o rows have `ocols` columns per head
 // (Dv, or Dv + 1 when the scan carried a column of ones).
-template <typename TO>
+template <typename TO, typename TG>
 __global__ void __launch_bounds__(256)
 scan_readout_kernel(const float* __restrict__ o, int ocols, const float* __restrict__ e, float den_eps, float oscale,
                     const float* __restrict__ skip, const float* __restrict__ x, long long ldx,
-                    const float* __restrict__ pre, long long ldpre, const float* __restrict__ post, long long ldpost,
+                    const float* __restrict__ pre, long long ldpre, const TG* __restrict__ post, long long ldpost,
                     int post_silu, const float* __restrict__ w, int w_full, TO* __restrict__ out, int H, int Dv, int groups, float eps) {
   extern __shared__ float row[];                         // [N] + [groups]
   const long long t = blockIdx.x;
@@ -581,7 +625,7 @@ scan_readout_kernel(const float* __restrict__ o, int ocols, const float* __restr
   __syncthreads();
   for (int c = threadIdx.x; c < N; c += blockDim.x) {
     float v = row[c] * gsum[c / GS] * w[w_full ? c : c % GS];
-    if (post) { const float z = post[t * ldpost + c]; v *= (post_silu ? z : 1.f) / (1.f + expf(-z)); }
+    if (post) { const float z = to_f32<TG>(post[t * ldpost + c]); v *= (post_silu ? z : 1.f) / (1.f + expf(-z)); }
     out[t * N + c] = from_f32<TO>(v);
   }
 }
@@ -672,12 +716,39 @@ B200_API int b200_short_conv_tail(const void* x, long long ldx, const float* in_
   return 0;
 }
 
+B200_API int b200_delta_gates_ex(float* q, long long ldq, float* k, long long ldk, float* a, long long lda, float* b, long long ldb,
+                                 const float* dt_bias, const float* A_log, int tokens, int G, int H, int D, int AD, float qscale,
+                                 float unit_eps, void* stream) {
+  using namespace b200;
+  if (tokens <= 0) return 0;
+  if (AD != D && AD != 1) return B200_ERR_BAD_SHAPE;
+  delta_gates_kernel<<<tokens, 128, 0, (cudaStream_t)stream>>>(q, ldq, k, ldk, a, lda, b, ldb, dt_bias, A_log, G, H, D, AD, qscale, unit_eps);
+  B200_LAUNCH_CHECK();
+  return 0;
+}
+
 B200_API int b200_delta_gates(float* q, long long ldq, float* k, long long ldk, float* a, long long lda, float* b, long long ldb,
                               const float* dt_bias, const float* A_log, int tokens, int G, int H, int D, float qscale,
                               float unit_eps, void* stream) {
+  return b200_delta_gates_ex(q, ldq, k, ldk, a, lda, b, ldb, dt_bias, A_log, tokens, G, H, D, D, qscale, unit_eps, stream);
+}
+
+B200_API int b200_token_shift(const void* h, long long ldh, const float* mu, float* prev, const int* pos, const int* slot, void* out,
+                              int tokens, int W, int S, int step_tail, int dtype, void* stream) {
   using namespace b200;
   if (tokens <= 0) return 0;
-  delta_gates_kernel<<<tokens, 128, 0, (cudaStream_t)stream>>>(q, ldq, k, ldk, a, lda, b, ldb, dt_bias, A_log, G, H, D, qscale, unit_eps);
+  if (W <= 0 || S <= 0) return B200_ERR_BAD_SHAPE;
+  cudaStream_t st = (cudaStream_t)stream;
+  const int es = dtype == B200_DT_FP32 ? 4 : 2;
+  const bool vec = W % 4 == 0 && ldh % 4 == 0 && !((reinterpret_cast<uintptr_t>(mu) | reinterpret_cast<uintptr_t>(prev)) & 15) &&
+                   !((reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(out)) & (4 * es - 1));
+  const long long n = (long long)tokens * (vec ? W / 4 : W);
+  const unsigned grid = (unsigned)((n + 255) / 256);
+#define SHIFT(TT, VV) token_shift_kernel<TT, VV><<<grid, 256, 0, st>>>((const TT*)h, ldh, mu, prev, pos, slot, (TT*)out, tokens, W, S, step_tail)
+  if (dtype == B200_DT_FP32) { if (vec) SHIFT(float, 4); else SHIFT(float, 1); }
+  else if (dtype == B200_DT_BF16) { if (vec) SHIFT(__nv_bfloat16, 4); else SHIFT(__nv_bfloat16, 1); }
+  else return B200_ERR_UNSUPPORTED;
+#undef SHIFT
   B200_LAUNCH_CHECK();
   return 0;
 }
@@ -688,7 +759,7 @@ B200_API int b200_linear_scan(const float* q, long long ldq, const float* k, lon
                               int mode, int act, int ones, void* stream) {
   using namespace b200;
   if (n_runs <= 0) return 0;
-  if (H <= 0 || G <= 0 || H % G || D <= 0 || Dv <= 0 || mode < 0 || mode > 2 || H > 65535 || ones < 0 || ones > 1 || Dv - ones < 1)
+  if (H <= 0 || G <= 0 || H % G || D <= 0 || Dv <= 0 || mode < 0 || mode > 3 || H > 65535 || ones < 0 || ones > 1 || Dv - ones < 1)
     return B200_ERR_BAD_SHAPE;
   // rows per thread R in {8, 16, 32}; lanes per column LPC = power of two with LPC * R >= D
   int R = D <= 8 ? 8 : (D <= 256 ? 16 : 32);
@@ -717,7 +788,8 @@ B200_API int b200_linear_scan(const float* q, long long ldq, const float* k, lon
   } while (0)
 #define SCAN(RR, LL)                                                                                                       \
   do {                                                                                                                     \
-    if (mode == 0) SCAN_K(RR, 0, LL); else if (mode == 1) SCAN_K(RR, 1, LL); else SCAN_K(RR, 2, LL);                       \
+    if (mode == 0) SCAN_K(RR, 0, LL); else if (mode == 1) SCAN_K(RR, 1, LL); else if (mode == 2) SCAN_K(RR, 2, LL);        \
+    else SCAN_K(RR, 3, LL);                                                                                                \
   } while (0)
   if (R == 8) SCAN(8, 1);
   else if (R == 16) {
@@ -762,9 +834,9 @@ B200_API int b200_ssm_gates(const float* dt, long long ld, const float* dt_bias,
 }
 
 B200_API int b200_scan_readout(const float* o, int ocols, const float* e, float den_eps, float oscale, const float* skip,
-                               const float* x, long long ldx, const float* pre, long long ldpre, const float* post,
-                               long long ldpost, int post_silu, const float* w, int w_full, void* out, long long tokens, int H, int Dv,
-                               int groups, float eps, int out_dtype, void* stream) {
+                               const float* x, long long ldx, const float* pre, long long ldpre, const void* post,
+                               long long ldpost, int post_silu, int post_dtype, const float* w, int w_full, void* out, long long tokens,
+                               int H, int Dv, int groups, float eps, int out_dtype, void* stream) {
   using namespace b200;
   if (tokens <= 0) return 0;
   if (H <= 0 || Dv <= 0 || groups <= 0 || (H * Dv) % groups || ocols < Dv || (e && ocols < Dv + 1) || (skip && !x))
@@ -772,15 +844,18 @@ B200_API int b200_scan_readout(const float* o, int ocols, const float* e, float 
   const size_t smem = ((size_t)H * Dv + groups) * sizeof(float);
   if (smem > 200 * 1024) return B200_ERR_TOO_LARGE;
   cudaStream_t st = (cudaStream_t)stream;
-#define READOUT(TO)                                                                                                          \
+#define READOUT(TO, TG)                                                                                                        \
   do {                                                                                                                       \
-    auto kern = scan_readout_kernel<TO>;                                                                                     \
+    auto kern = scan_readout_kernel<TO, TG>;                                                                                 \
     if (smem > 48 * 1024) B200_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));    \
-    kern<<<(unsigned)tokens, 256, smem, st>>>(o, ocols, e, den_eps, oscale, skip, x, ldx, pre, ldpre, post, ldpost, post_silu, w, w_full,  \
+    kern<<<(unsigned)tokens, 256, smem, st>>>(o, ocols, e, den_eps, oscale, skip, x, ldx, pre, ldpre, (const TG*)post, ldpost, post_silu, w, w_full,  \
                                               (TO*)out, H, Dv, groups, eps);                                                 \
   } while (0)
-  if (out_dtype == B200_DT_FP32) READOUT(float);
-  else if (out_dtype == B200_DT_BF16) READOUT(__nv_bfloat16);
+  const bool gate16 = post && post_dtype == B200_DT_BF16;
+  if (gate16 && out_dtype == B200_DT_BF16) READOUT(__nv_bfloat16, __nv_bfloat16);
+  else if (gate16) return B200_ERR_UNSUPPORTED;
+  else if (out_dtype == B200_DT_FP32) READOUT(float, float);
+  else if (out_dtype == B200_DT_BF16) READOUT(__nv_bfloat16, float);
   else return B200_ERR_UNSUPPORTED;
 #undef READOUT
   B200_LAUNCH_CHECK();

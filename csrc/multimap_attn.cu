@@ -4,13 +4,16 @@
 //   keys    cache K [blocks, G * M, block_size, D]   (key head g, map m at row g * M + m; normed and rotated when stored)
 //   values  cache V [blocks, G,     block_size, Dv]  (Dv need not equal D)
 //   token t (position p of cache row slot[t]) sees key j of its row if j <= p and (p - j < window or j < keep_first);
-//   window <= 0 means every j <= p.
+//   window <= 0 means every j <= p; opts.chunk > 0 (instead of a window): only keys of p's own chunk, j / chunk == p / chunk.
 //   a_m = softmax_j(scale q_{h,m} . k_{g,m,j}) V_g        g = h / (H / G)
 //   M = 2, combine:  o = a_0 - lambda a_1 ;  o <- o / sqrt(mean(o^2) + eps) * post      (differential attention)
 //   otherwise:       o = a_0 post (M = 1)
+//   b200_attn_opts (one map, every field optional): scores pass cap tanh(s / cap) before the softmax; a number per head whose
+//   exponential joins the softmax's denominator (a sink: no key, no value); o_h times sigmoid(gate[t, h]).
 //
-// b200_qknorm_rope_store   per-(head, map) RMS norm with a weight over D, rotary on the first `rot` dims in the split layout
-//                          (dim i pairs with i + rot/2), q -> q_out in the cache dtype, k and v -> their pages.
+// b200_qkv_store           bias, per-(head, map) RMS norm with a weight over D (or none), rotary on the first `rot` dims in the split
+//                          layout (dim i pairs with i + rot/2), values mixed with those another layer cached for the same token;
+//                          q -> q_out in the cache dtype, k and v -> their pages. b200_qknorm_rope_store: its fp32 subset.
 // b200_conv_qknorm_store   what stands in front of one-map attention whose projections pass a short causal convolution: bias,
 //                          convolution over time on every channel of q | k | v (inputs before the run come from a carried tail),
 //                          per-row RMS norm without a weight (v optional), q times a factor that grows with the position.
@@ -20,6 +23,8 @@
 //                          (a warp per (token, head)) for row sizes that are not whole chunks.
 #include "common.cuh"
 #include "mma_sync.cuh"
+
+#include <type_traits>
 #include "../include/b200_ops.h"
 
 #define B200_DISPATCH_T(dtype, ...)                                   \
@@ -30,54 +35,135 @@
 
 namespace b200 {
 
-// proj fp32 [tokens, ld]: q rows (QR = H * M of D) at column 0, then (has_kv) k rows (KR = G * M of D) and v (G * Dv).
-template <typename T>
-__global__ void __launch_bounds__(128)
-qknorm_rope_store_kernel(const float* __restrict__ proj, long long ld, const float* __restrict__ wq, const float* __restrict__ wk,
-                         const float* __restrict__ cs, const float* __restrict__ sn, const int* __restrict__ pos,
-                         const int* __restrict__ slot, const int* __restrict__ table, int max_blocks, T* __restrict__ q_out,
-                         T* __restrict__ ck, T* __restrict__ cv, int QR, int KR, int G, int D, int Dv, int rot, int block_size,
-                         float eps, int has_kv) {
-  extern __shared__ float sh[];                          // [warps, D]
-  const int t = blockIdx.x;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-  const int p = pos[t];
-  const float* row = proj + (long long)t * ld;
-  const float* c = cs + (long long)p * (rot / 2);
-  const float* s = sn + (long long)p * (rot / 2);
-  float* buf = sh + warp * D;
-  long long kbase = 0, vbase = 0;
-  if (has_kv) {
-    const int blk = table[(long long)slot[t] * max_blocks + p / block_size];
-    const int off = p % block_size;
-    kbase = ((long long)blk * KR * block_size + off) * D;            // + r * block_size * D
-    vbase = ((long long)blk * G * block_size + off) * Dv;            // + g * block_size * Dv
+// proj [tokens, ld]: q rows (QR = H * M of D) at column 0, then (has_kv) k rows (KR = G * M of D) and v (G rows of Dv). A warp
+// owns one of these rows over TB consecutive tokens. A row is walked as pairs: (i, i + rot / 2) inside the rotated part and
+// (i, i + half of the rest) behind it, so every lane has both members of the pairs it turns; V pairs lie next to each other,
+// a lane owns up to NI groups of them, their biases and norm weights stay in registers. Rows of v (and of a layer without
+// rotation) are one unrotated part.
+struct QkvStoreArgs {
+  const void* proj; long long ld;
+  const float *bias, *wq, *wk;                           // bias [QR D + KR D + G Dv] or NULL; wq NULL: rows are not normed
+  const float *cs, *sn;                                  // [max_pos, rot / 2]
+  const int *pos, *slot, *table;
+  void *q_out, *ck, *cv;
+  const void* v_first; const float* v_lambda;            // v <- (1 - lambda) v + lambda v_first at the token's place in that pool
+  int max_blocks, tokens, QR, KR, G, D, Dv, rot, block_size, has_kv, TB;
+  float eps;
+};
+
+template <typename TX, int V> __device__ __forceinline__ void load_v(const TX* p, float (&v)[V]) {
+  if (V == 2 && std::is_same<TX, __nv_bfloat16>::value) {
+    const float2 f = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(p));
+    v[0] = f.x; v[V - 1] = f.y;
+  } else if (V == 2 && sizeof(TX) == 4) {
+    const float2 f = *reinterpret_cast<const float2*>(p);
+    v[0] = f.x; v[V - 1] = f.y;
+  } else {
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] = to_f32<TX>(p[e]);
   }
-  const int rows = QR + (has_kv ? KR : 0);
-  const int hr = rot / 2;
-  for (int r = warp; r < rows; r += nw) {
-    const float* x = row + (long long)r * D;
-    const float* w = r < QR ? wq : wk;
-    float ss = 0.f;
-    for (int d = lane; d < D; d += 32) { const float v = x[d]; ss += v * v; }
-    ss = warp_sum(ss);
-    const float sc = rsqrtf(ss / D + eps);
-    __syncwarp();
-    for (int d = lane; d < D; d += 32) buf[d] = x[d] * sc * w[d];
-    __syncwarp();
-    T* dst = r < QR ? q_out + ((long long)t * QR + r) * D : ck + kbase + (long long)(r - QR) * block_size * D;
-    for (int d = lane; d < D; d += 32) {
-      float v = buf[d];
-      if (d < hr) v = buf[d] * c[d] - buf[d + hr] * s[d];
-      else if (d < rot) v = buf[d] * c[d - hr] + buf[d - hr] * s[d - hr];
-      dst[d] = from_f32<T>(v);
+}
+template <typename T, int V> __device__ __forceinline__ void store_v(T* p, const float (&v)[V]) {
+  if (V == 2 && std::is_same<T, __nv_bfloat16>::value) *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(v[0], v[V - 1]);
+  else if (V == 2 && sizeof(T) == 4) *reinterpret_cast<float2*>(p) = make_float2(v[0], v[V - 1]);
+  else {
+#pragma unroll
+    for (int e = 0; e < V; ++e) p[e] = from_f32<T>(v[e]);
+  }
+}
+
+template <typename TX, typename T, int V, int NI>
+__global__ void __launch_bounds__(128)
+qkv_store_kernel(const QkvStoreArgs a) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int r = blockIdx.y * 4 + warp;
+  if (r >= a.QR + (a.has_kv ? a.KR + a.G : 0)) return;
+  const bool is_q = r < a.QR, is_v = r >= a.QR + a.KR;
+  const int RS = is_v ? a.Dv : a.D;
+  const int col0 = is_v ? (a.QR + a.KR) * a.D + (r - a.QR - a.KR) * a.Dv : r * a.D;
+  const int hr = is_v ? 0 : a.rot / 2;
+  const int ph = (RS - 2 * hr + 1) / 2;                  // pairs behind the rotated part
+  const float* w = is_v || !a.wq ? nullptr : (is_q ? a.wq : a.wk);
+  int i0[NI], i1[NI];                                    // first member of a group of pairs, and how far the second lies; < 0: none
+  float b0[NI][V], b1[NI][V], w0[NI][V], w1[NI][V];
+#pragma unroll
+  for (int i = 0; i < NI; ++i) {
+    const int x = (lane + 32 * i) * V;
+    if (x < hr) { i0[i] = x; i1[i] = x + hr; }
+    else if (x < hr + ph) { i0[i] = x + hr; i1[i] = x + hr + ph < RS ? x + hr + ph : -1; }
+    else i0[i] = i1[i] = -1;
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      b0[i][e] = a.bias && i0[i] >= 0 ? a.bias[col0 + i0[i] + e] : 0.f;
+      b1[i][e] = a.bias && i1[i] >= 0 ? a.bias[col0 + i1[i] + e] : 0.f;
+      w0[i][e] = w && i0[i] >= 0 ? w[i0[i] + e] : 1.f;
+      w1[i][e] = w && i1[i] >= 0 ? w[i1[i] + e] : 1.f;
     }
   }
-  if (has_kv) {
-    const float* vsrc = row + (long long)(QR + KR) * D;
-    for (int i = threadIdx.x; i < G * Dv; i += blockDim.x) {
-      const int g = i / Dv, d = i % Dv;
-      cv[vbase + (long long)g * block_size * Dv + d] = from_f32<T>(vsrc[i]);
+  const float lam = is_v && a.v_first ? a.v_lambda[0] : 0.f;
+  const int t0 = blockIdx.x * a.TB, t1 = min(a.tokens, t0 + a.TB);
+  for (int t = t0; t < t1; ++t) {
+    const int p = a.pos[t];
+    const TX* src = reinterpret_cast<const TX*>(a.proj) + (long long)t * a.ld + col0;
+    float x0[NI][V], x1[NI][V], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+#pragma unroll
+      for (int e = 0; e < V; ++e) x0[i][e] = x1[i][e] = 0.f;
+      if (i0[i] >= 0) load_v<TX, V>(src + i0[i], x0[i]);
+      if (i1[i] >= 0) load_v<TX, V>(src + i1[i], x1[i]);
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        x0[i][e] += b0[i][e];
+        x1[i][e] += b1[i][e];
+        ss = fmaf(x0[i][e], x0[i][e], ss);
+        ss = fmaf(x1[i][e], x1[i][e], ss);
+      }
+    }
+    if (w) {
+      const float f = rsqrtf(warp_sum(ss) / RS + a.eps);
+#pragma unroll
+      for (int i = 0; i < NI; ++i)
+#pragma unroll
+        for (int e = 0; e < V; ++e) { x0[i][e] *= f * w0[i][e]; x1[i][e] *= f * w1[i][e]; }
+    }
+    T* dst;
+    long long place = 0;
+    if (is_q) dst = reinterpret_cast<T*>(a.q_out) + ((long long)t * a.QR + r) * a.D;
+    else {
+      const long long blk = a.table[(long long)a.slot[t] * a.max_blocks + p / a.block_size];
+      const int off = p % a.block_size;
+      if (is_v) place = ((blk * a.G + (r - a.QR - a.KR)) * a.block_size + off) * a.Dv;
+      else place = ((blk * a.KR + (r - a.QR)) * a.block_size + off) * a.D;
+      dst = reinterpret_cast<T*>(is_v ? a.cv : a.ck) + place;
+    }
+    const float* c = a.cs + (long long)p * hr;
+    const float* s = a.sn + (long long)p * hr;
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int x = (lane + 32 * i) * V;
+      if (x < hr) {
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+          const float u = x0[i][e], v = x1[i][e], cc = c[x + e], sn = s[x + e];
+          x0[i][e] = u * cc - v * sn;
+          x1[i][e] = v * cc + u * sn;
+        }
+      } else if (is_v && a.v_first) {
+        const T* vf = reinterpret_cast<const T*>(a.v_first) + place;
+        float f0[V], f1[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) f0[e] = f1[e] = 0.f;
+        if (i0[i] >= 0) load_v<T, V>(vf + i0[i], f0);
+        if (i1[i] >= 0) load_v<T, V>(vf + i1[i], f1);
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+          x0[i][e] = (1.f - lam) * x0[i][e] + lam * f0[e];
+          x1[i][e] = (1.f - lam) * x1[i][e] + lam * f1[e];
+        }
+      }
+      if (i0[i] >= 0) store_v<T, V>(dst + i0[i], x0[i]);
+      if (i1[i] >= 0) store_v<T, V>(dst + i1[i], x1[i]);
     }
   }
 }
@@ -200,6 +286,16 @@ conv_qknorm_store_kernel(const TX* __restrict__ proj, long long ld, const float*
 }
 
 constexpr int kMaxDv = 256;
+constexpr float kLog2e = 1.4426950408889634f;
+
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+// the first key position p sees besides kept ones: the window's lower edge, or the start of p's chunk
+__device__ __forceinline__ int first_seen(int p, int window, int chunk) {
+  if (chunk > 0) return p / chunk * chunk;
+  return window > 0 && p + 1 - window > 0 ? p + 1 - window : 0;
+}
+template <typename T> __device__ __forceinline__ float capped_tanh(float x) { return tanh_ex2(x); }
+template <> __device__ __forceinline__ float capped_tanh<float>(float x) { return tanhf(x); }
 constexpr int kAcc = kMaxDv / 32;
 constexpr int kMaxMaps = 2;
 
@@ -234,7 +330,7 @@ __global__ void __launch_bounds__(128)
 multimap_attn_kernel(const T* __restrict__ q, const T* __restrict__ ck, const T* __restrict__ cv, const int* __restrict__ pos,
                      const int* __restrict__ slot, const int* __restrict__ table, int max_blocks, T* __restrict__ out, long long ldo, int tokens,
                      int H, int G, int M, int D, int Dv, int block_size, float scale, int window, int keep_first, int combine,
-                     float lambda, float post, float eps) {
+                     float lambda, float post, float eps, const b200_attn_opts opt) {
   extern __shared__ float qs[];                          // [warps, D]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const long long item = (long long)blockIdx.x * nw + warp;          // (token, head)
@@ -243,9 +339,8 @@ multimap_attn_kernel(const T* __restrict__ q, const T* __restrict__ ck, const T*
   const int g = h / (H / G);
   const int p = pos[t];
   const int* trow = table + (long long)slot[t] * max_blocks;
-  int lo = 0;
-  if (window > 0 && p + 1 - window > 0) lo = p + 1 - window;
-  const int n1 = min(max(keep_first, 0), lo);            // kept first tokens that the window no longer covers
+  const int lo = first_seen(p, window, opt.chunk);
+  const int n1 = window > 0 ? min(max(keep_first, 0), lo) : 0;       // kept first tokens that the window no longer covers
   const int total = n1 + (p + 1 - lo);
   float* myq = qs + warp * D;
   float res[kAcc];
@@ -271,6 +366,7 @@ multimap_attn_kernel(const T* __restrict__ q, const T* __restrict__ ck, const T*
         const int blk = trow[kp / block_size];
         const int off = kp % block_size;
         sc = dot_qk<T>(myq, ck + (((long long)blk * G * M + kh) * block_size + off) * D, D) * scale;
+        if (opt.softcap > 0.f) sc = opt.softcap * capped_tanh<T>(sc / opt.softcap);
         voff = (((long long)blk * G + g) * block_size + off) * Dv;
       }
       const float m_new = fmaxf(mx, warp_max(sc));
@@ -292,6 +388,7 @@ multimap_attn_kernel(const T* __restrict__ q, const T* __restrict__ ck, const T*
         }
       }
     }
+    if (opt.sink) l += expf(opt.sink[h] - mx);
     const float inv = l > 0.f ? 1.f / l : 0.f;
     const float coef = (m == 0) ? 1.f : -lambda;
 #pragma unroll
@@ -305,6 +402,7 @@ multimap_attn_kernel(const T* __restrict__ q, const T* __restrict__ ck, const T*
     ss = warp_sum(ss);
     mult = rsqrtf(ss / Dv + eps) * post;
   }
+  if (opt.gate) mult *= sigmoid_f(opt.gate[(long long)t * opt.ld_gate + h]);
   T* orow = out + (long long)t * ldo + (long long)h * Dv;
 #pragma unroll
   for (int a = 0; a < kAcc; ++a) {
@@ -326,7 +424,7 @@ __global__ void __launch_bounds__(128, 4)               // four CTAs per SM: a d
 multimap_attn_vec_kernel(const T* __restrict__ q, const T* __restrict__ ck, const T* __restrict__ cv, const int* __restrict__ pos,
                          const int* __restrict__ slot, const int* __restrict__ table, int max_blocks, T* __restrict__ out, long long ldo,
                          float* __restrict__ part, int H, int G, int M, int D, int Dv, int bs_log2, float scale, int window,
-                         int keep_first, int nsplit, float post, int CP, int CPK, int CPV) {
+                         int keep_first, int nsplit, float post, int CP, int CPK, int CPV, const b200_attn_opts opt) {
   constexpr int E = 16 / sizeof(T);
   extern __shared__ float sm[];                          // [4 warps][HB][Dv + 2]
   const int t = blockIdx.x;
@@ -345,9 +443,8 @@ multimap_attn_vec_kernel(const T* __restrict__ q, const T* __restrict__ ck, cons
   for (int x = 0; x < VC; ++x) liveV[x] = c + x * CP < CPV;
   const int p = pos[t];
   const int* trow = table + (long long)slot[t] * max_blocks;
-  int lo = 0;
-  if (window > 0 && p + 1 - window > 0) lo = p + 1 - window;
-  const int n1 = min(max(keep_first, 0), lo);
+  const int lo = first_seen(p, window, opt.chunk);
+  const int n1 = window > 0 ? min(max(keep_first, 0), lo) : 0;
   const int total = n1 + (p + 1 - lo);
   int i_lo = 0, i_hi = total;
   if (nsplit > 1) {
@@ -357,7 +454,10 @@ multimap_attn_vec_kernel(const T* __restrict__ q, const T* __restrict__ ck, cons
   }
   // scores are kept in units of log 2 (scale * log2(e) is folded into q): one ex2 per exponential; the merge kernel reads
   // the recorded maxima in the same units
-  const float sl2 = scale * 1.4426950408889634f;
+  // (with a cap: q . k scale / cap leaves the product, and cap log2(e) multiplies its tanh)
+  const bool capped = opt.softcap > 0.f;
+  const float sl2 = capped ? scale / opt.softcap : scale * kLog2e;
+  const float cap2 = opt.softcap * kLog2e;
   float qv[HB][E], acc[HB][VC][E], mx[HB], l[HB];
 #pragma unroll
   for (int hh = 0; hh < HB; ++hh) {
@@ -414,6 +514,7 @@ multimap_attn_vec_kernel(const T* __restrict__ q, const T* __restrict__ ck, cons
 #pragma unroll
         for (int e = 0; e < E; ++e) s = fmaf(qv[hh][e], kf[e], s);
         for (int o = CP >> 1; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+        if (capped) s = cap2 * capped_tanh<T>(s);
         sc[u][hh] = valid[u] ? s : -INFINITY;
       }
     }
@@ -490,7 +591,10 @@ multimap_attn_vec_kernel(const T* __restrict__ q, const T* __restrict__ ck, cons
       }
     }
     if (direct) {
-      out[(long long)t * ldo + (long long)h * Dv + d] = from_f32<T>(lt > 0.f ? at / lt * post : 0.f);
+      float f = post;
+      if (opt.sink) lt += exp2f(opt.sink[h] * kLog2e - mt);
+      if (opt.gate) f *= sigmoid_f(opt.gate[(long long)t * opt.ld_gate + h]);
+      out[(long long)t * ldo + (long long)h * Dv + d] = from_f32<T>(lt > 0.f ? at / lt * f : 0.f);
     } else {
       float* pr = part + ((((long long)t * H + h) * M + m) * nsplit + split) * LDW;
       if (d == 0) { pr[0] = mt; pr[1] = lt; }
@@ -503,7 +607,7 @@ multimap_attn_vec_kernel(const T* __restrict__ q, const T* __restrict__ ck, cons
 template <typename T>
 __global__ void __launch_bounds__(128)
 multimap_attn_merge_kernel(const float* __restrict__ part, T* __restrict__ out, long long ldo, int H, long long items, int M, int Dv, int nsplit,
-                           int combine, float lambda, float post, float eps) {
+                           int combine, float lambda, float post, float eps, const b200_attn_opts opt) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long long item = (long long)blockIdx.x * 4 + warp;            // (token, head)
   if (item >= items) return;
@@ -529,6 +633,7 @@ multimap_attn_merge_kernel(const float* __restrict__ part, T* __restrict__ out, 
         if (d < Dv) at[a] += pr[s * LDW + 2 + d] * e;
       }
     }
+    if (opt.sink) lt += exp2f(opt.sink[item % H] * kLog2e - mt);
     const float inv = lt > 0.f ? 1.f / lt : 0.f;
     const float coef = m == 0 ? 1.f : -lambda;
 #pragma unroll
@@ -542,6 +647,7 @@ multimap_attn_merge_kernel(const float* __restrict__ part, T* __restrict__ out, 
     ss = warp_sum(ss);
     mult = rsqrtf(ss / Dv + eps) * post;
   }
+  if (opt.gate) mult *= sigmoid_f(opt.gate[item / H * opt.ld_gate + item % H]);
 #pragma unroll
   for (int a = 0; a < kAcc; ++a) {
     const int d = lane + 32 * a;
@@ -550,20 +656,53 @@ multimap_attn_merge_kernel(const float* __restrict__ part, T* __restrict__ out, 
 }
 }  // namespace b200
 
+B200_API int b200_qkv_store(const void* proj, long long ld, const float* bias, const float* wq, const float* wk, const float* cos_t,
+                            const float* sin_t, const int* pos, const int* slot, const int* table, int max_blocks, void* q_out,
+                            void* ck, void* cv, const void* v_first, const float* v_lambda, int tokens, int H, int G, int M, int D,
+                            int Dv, int rot, int block_size, float eps, int has_kv, int x_dtype, int dtype, void* stream) {
+  using namespace b200;
+  if (tokens <= 0) return 0;
+  if (H <= 0 || G <= 0 || M <= 0 || D <= 0 || rot < 0 || rot > D || (rot & 1) || block_size <= 0 || (has_kv && Dv <= 0)) return B200_ERR_BAD_SHAPE;
+  if ((wq && has_kv && !wk) || (v_first && (!v_lambda || !has_kv)) || (rot && (!cos_t || !sin_t))) return B200_ERR_BAD_SHAPE;
+  const int big = has_kv && Dv > D ? Dv : D;
+  if (big > 512) return B200_ERR_TOO_LARGE;
+  const int es = x_dtype == B200_DT_FP32 ? 4 : 2, eo = dtype == B200_DT_FP32 ? 4 : 2;
+  auto al = [](const void* p_, int n) { return !(reinterpret_cast<uintptr_t>(p_) & (n - 1)); };
+  // two neighbouring pairs per lane: both parts of a row, and where their second halves start, are even
+  const bool v2 = D % 4 == 0 && rot % 4 == 0 && (!has_kv || Dv % 4 == 0) && ld % 2 == 0 && al(proj, 2 * es) && al(q_out, 2 * eo) &&
+                  (!has_kv || (al(ck, 2 * eo) && al(cv, 2 * eo))) && (!v_first || al(v_first, 2 * eo));
+  QkvStoreArgs a;
+  a.proj = proj; a.ld = ld; a.bias = bias; a.wq = wq; a.wk = wk; a.cs = cos_t; a.sn = sin_t; a.pos = pos; a.slot = slot; a.table = table;
+  a.q_out = q_out; a.ck = ck; a.cv = cv; a.v_first = v_first; a.v_lambda = v_lambda; a.max_blocks = max_blocks; a.tokens = tokens;
+  a.QR = H * M; a.KR = G * M; a.G = G; a.D = D; a.Dv = Dv; a.rot = rot; a.block_size = block_size; a.has_kv = has_kv; a.eps = eps;
+  a.TB = tokens <= 512 ? 1 : 8;
+  const dim3 grid((tokens + a.TB - 1) / a.TB, (a.QR + (has_kv ? a.KR + G : 0) + 3) / 4);
+  if (grid.y > 65535) return B200_ERR_TOO_LARGE;
+  cudaStream_t st = (cudaStream_t)stream;
+#define QS(TX, T, VV, NN) qkv_store_kernel<TX, T, VV, NN><<<grid, 128, 0, st>>>(a)
+  // pairs of a row: at most big / 2 + 1
+#define QS_V(TX, T)                                                                                                          \
+  do {                                                                                                                       \
+    if (v2 && big <= 128) QS(TX, T, 2, 1); else if (v2 && big <= 256) QS(TX, T, 2, 2); else if (v2) QS(TX, T, 2, 4);           \
+    else if (big <= 62) QS(TX, T, 1, 1); else if (big <= 126) QS(TX, T, 1, 2); else QS(TX, T, 1, 9);                          \
+  } while (0)
+  if (x_dtype == B200_DT_FP32 && dtype == B200_DT_FP32) QS_V(float, float);
+  else if (x_dtype == B200_DT_FP32 && dtype == B200_DT_BF16) QS_V(float, __nv_bfloat16);
+  else if (x_dtype == B200_DT_FP32 && dtype == B200_DT_FP16) QS_V(float, __half);
+  else if (x_dtype == B200_DT_BF16 && dtype == B200_DT_BF16) QS_V(__nv_bfloat16, __nv_bfloat16);
+  else return B200_ERR_UNSUPPORTED;
+#undef QS_V
+#undef QS
+  B200_LAUNCH_CHECK();
+  return 0;
+}
+
 B200_API int b200_qknorm_rope_store(const float* proj, long long ld, const float* wq, const float* wk, const float* cos_t,
                                     const float* sin_t, const int* pos, const int* slot, const int* table, int max_blocks,
                                     void* q_out, void* ck, void* cv, int tokens, int H, int G, int M, int D, int Dv, int rot,
                                     int block_size, float eps, int has_kv, int dtype, void* stream) {
-  using namespace b200;
-  if (tokens <= 0) return 0;
-  if (H <= 0 || G <= 0 || M <= 0 || D <= 0 || rot < 0 || rot > D || (rot & 1) || block_size <= 0) return B200_ERR_BAD_SHAPE;
-  const size_t smem = 4 * (size_t)D * 4;
-  if (smem > 48 * 1024) return B200_ERR_TOO_LARGE;
-  B200_DISPATCH_T(dtype, qknorm_rope_store_kernel<T><<<tokens, 128, smem, (cudaStream_t)stream>>>(
-      proj, ld, wq, wk, cos_t, sin_t, pos, slot, table, max_blocks, (T*)q_out, (T*)ck, (T*)cv, H * M, G * M, G, D, Dv, rot,
-      block_size, eps, has_kv));
-  B200_LAUNCH_CHECK();
-  return 0;
+  return b200_qkv_store(proj, ld, nullptr, wq, wk, cos_t, sin_t, pos, slot, table, max_blocks, q_out, ck, cv, nullptr, nullptr, tokens, H,
+                        G, M, D, Dv, rot, block_size, eps, has_kv, B200_DT_FP32, dtype, stream);
 }
 
 B200_API int b200_conv_qknorm_store(const void* proj, long long ld, const float* bias, const float* w, const float* tail, const int* pos,
@@ -605,12 +744,14 @@ B200_API int b200_conv_qknorm_store(const void* proj, long long ld, const float*
   return 0;
 }
 
-B200_API int b200_multimap_attn(const void* q, const void* ck, const void* cv, const int* pos, const int* slot, const int* table,
-                                int max_blocks, void* out, long long ldo, float* part, int tokens, int H, int G, int M, int D, int Dv,
-                                int block_size, float scale, int window, int keep_first, int nsplit, int combine, float lambda,
-                                float post, float eps, int dtype, void* stream) {
+B200_API int b200_multimap_attn_ex(const void* q, const void* ck, const void* cv, const int* pos, const int* slot, const int* table,
+                                   int max_blocks, void* out, long long ldo, float* part, int tokens, int H, int G, int M, int D, int Dv,
+                                   int block_size, float scale, int window, int keep_first, int nsplit, int combine, float lambda,
+                                   float post, float eps, const b200_attn_opts* opts, int dtype, void* stream) {
   using namespace b200;
   if (tokens <= 0) return 0;
+  const b200_attn_opts opt = opts ? *opts : b200_attn_opts{};
+  if (opts && (M != 1 || opt.chunk < 0 || (opt.chunk > 0 && window > 0) || !(opt.softcap >= 0.f))) return B200_ERR_UNSUPPORTED;
   if (H <= 0 || G <= 0 || H % G || M < 1 || M > kMaxMaps || D <= 0 || Dv <= 0 || block_size <= 0 || nsplit < 1) return B200_ERR_BAD_SHAPE;
   if (Dv > kMaxDv) return B200_ERR_TOO_LARGE;
   if (combine && M != 2) return B200_ERR_UNSUPPORTED;
@@ -637,7 +778,7 @@ B200_API int b200_multimap_attn(const void* q, const void* ck, const void* cv, c
       const size_t smem = (size_t)4 * HB * (Dv + 2) * sizeof(float);
 #define MMV2(T, HBV, VCV)                                                                                                    \
   multimap_attn_vec_kernel<T, HBV, VCV><<<grid, 128, smem, st>>>((const T*)q, (const T*)ck, (const T*)cv, pos, slot, table,   \
-      max_blocks, (T*)out, ldo, part, H, G, M, D, Dv, bs_log2, scale, window, keep_first, nsplit, post, CP, CPK, CPV)
+      max_blocks, (T*)out, ldo, part, H, G, M, D, Dv, bs_log2, scale, window, keep_first, nsplit, post, CP, CPK, CPV, opt)
 #define MMV(T, HBV)                                                                                                          \
   do { if (VC == 2) MMV2(T, HBV, 2); else MMV2(T, HBV, 1); } while (0)
 #define MMV_T(T)                                                                                                             \
@@ -645,7 +786,7 @@ B200_API int b200_multimap_attn(const void* q, const void* ck, const void* cv, c
     if (HB == 4) MMV(T, 4); else if (HB == 2) MMV(T, 2); else MMV(T, 1);                                                     \
     if (!direct)                                                                                                             \
       multimap_attn_merge_kernel<T><<<(unsigned)(((long long)tokens * H + 3) / 4), 128, 0, st>>>(                             \
-          part, (T*)out, ldo, H, (long long)tokens * H, M, Dv, nsplit, combine, lambda, post, eps);                                  \
+          part, (T*)out, ldo, H, (long long)tokens * H, M, Dv, nsplit, combine, lambda, post, eps, opt);                             \
   } while (0)
       if (dtype == B200_DT_BF16) MMV_T(__nv_bfloat16);
       else if (dtype == B200_DT_FP16) MMV_T(__half);
@@ -664,7 +805,15 @@ B200_API int b200_multimap_attn(const void* q, const void* ck, const void* cv, c
   const unsigned grid = (unsigned)(((long long)tokens * H + nw - 1) / nw);
   B200_DISPATCH_T(dtype, multimap_attn_kernel<T><<<grid, nw * 32, smem, st>>>(
       (const T*)q, (const T*)ck, (const T*)cv, pos, slot, table, max_blocks, (T*)out, ldo, tokens, H, G, M, D, Dv, block_size, scale,
-      window, keep_first, combine, lambda, post, eps));
+      window, keep_first, combine, lambda, post, eps, opt));
   B200_LAUNCH_CHECK();
   return 0;
+}
+
+B200_API int b200_multimap_attn(const void* q, const void* ck, const void* cv, const int* pos, const int* slot, const int* table,
+                                int max_blocks, void* out, long long ldo, float* part, int tokens, int H, int G, int M, int D, int Dv,
+                                int block_size, float scale, int window, int keep_first, int nsplit, int combine, float lambda,
+                                float post, float eps, int dtype, void* stream) {
+  return b200_multimap_attn_ex(q, ck, cv, pos, slot, table, max_blocks, out, ldo, part, tokens, H, G, M, D, Dv, block_size, scale, window,
+                               keep_first, nsplit, combine, lambda, post, eps, nullptr, dtype, stream);
 }

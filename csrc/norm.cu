@@ -426,12 +426,13 @@ B200_API int b200_norm_bwd_noalloc(int layer_norm, const void* dy, const void* h
 // ---------------------------------------------------------------------------------------------
 namespace b200 {
 // `center` 1: both norms take the row's mean off first and divide by the root of the variance (a layer norm with a weight and
-// no bias); the statistics are two passes over the row in shared memory (mean, then squared deviations).
+// no bias); the statistics are two passes over the row in shared memory (mean, then squared deviations). `y2`: a second branch
+// with a weight of its own, normed by itself and added to the first.
 template <typename TY, typename TH, typename WT>
 __global__ void __launch_bounds__(kNormThreads)
-sandwich_norm_kernel(const TY* __restrict__ y, const WT* __restrict__ w_post, const float* __restrict__ res_in,
-                     float* __restrict__ res_out, const WT* __restrict__ w_next, TH* __restrict__ h, int cols, float eps,
-                     float off, float mult, int center) {
+sandwich_norm_kernel(const TY* __restrict__ y, const WT* __restrict__ w_post, const TY* __restrict__ y2,
+                     const WT* __restrict__ w_post2, const float* __restrict__ res_in, float* __restrict__ res_out, const WT* __restrict__ w_next, TH* __restrict__ h,
+                     int cols, float eps, float off, float mult, int center) {
   extern __shared__ float rowbuf[];
   __shared__ float red[32];
   const long long row = blockIdx.x;
@@ -457,11 +458,24 @@ sandwich_norm_kernel(const TY* __restrict__ y, const WT* __restrict__ w_post, co
     ss = block_sum(ss, red);
     r1 = 1.f / sqrtf(ss / (float)cols + eps);
   }
+  float* rowbuf2 = rowbuf + cols;                       // y2 only
+  float r3 = 1.f;
+  if (y2) {
+    float s3 = 0.f;
+    for (int i = threadIdx.x; i < cols; i += blockDim.x) {
+      const float v = to_f32<TY>(y2[row * cols + i]);
+      rowbuf2[i] = v;
+      s3 += v * v;
+    }
+    s3 = block_sum(s3, red);
+    r3 = 1.f / sqrtf(s3 / (float)cols + eps);
+  }
   __syncthreads();
   float s2 = 0.f, t1 = 0.f;
   for (int i = threadIdx.x; i < cols; i += blockDim.x) {
     float v = rowbuf[i];
     if (w_post) v = (v - m1) * r1 * (off + to_f32<WT>(w_post[i]));
+    if (y2) v = fmaf(rowbuf2[i] * r3, off + to_f32<WT>(w_post2[i]), v);
     v *= mult;
     if (res_in) v += res_in[row * cols + i];
     rowbuf[i] = v;
@@ -487,15 +501,15 @@ sandwich_norm_kernel(const TY* __restrict__ y, const WT* __restrict__ w_post, co
 }
 
 template <typename TY, typename TH, typename WT>
-static int sandwich_launch(const void* y, const void* w_post, const float* res_in, float* res_out, const void* w_next, void* h,
-                           long long rows, int cols, float eps, float off, float mult, int center, cudaStream_t st) {
-  const size_t smem = (size_t)cols * sizeof(float);
+static int sandwich_launch(const void* y, const void* w_post, const void* y2, const void* w_post2, const float* res_in, float* res_out,
+                           const void* w_next, void* h, long long rows, int cols, float eps, float off, float mult, int center, cudaStream_t st) {
+  const size_t smem = (size_t)cols * (y2 ? 2 : 1) * sizeof(float);
   auto kern = sandwich_norm_kernel<TY, TH, WT>;
   if (smem > 48 * 1024) {
     if (smem > 200 * 1024) return B200_ERR_TOO_LARGE;
     B200_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   }
-  kern<<<(unsigned)rows, kNormThreads, smem, st>>>((const TY*)y, (const WT*)w_post, res_in, res_out, (const WT*)w_next, (TH*)h,
+  kern<<<(unsigned)rows, kNormThreads, smem, st>>>((const TY*)y, (const WT*)w_post, (const TY*)y2, (const WT*)w_post2, res_in, res_out, (const WT*)w_next, (TH*)h,
                                                    cols, eps, off, mult, center);
   B200_LAUNCH_CHECK();
   return 0;
@@ -541,15 +555,15 @@ poly_norm_kernel(const T* __restrict__ z, const float* __restrict__ act, T* __re
 }
 }  // namespace b200
 
-B200_API int b200_sandwich_norm_c(const void* y, const void* w_post, const float* res_in, float* res_out, const void* w_next,
-                                  void* h, long long rows, int cols, float eps, float off, float mult, int center, int y_dtype,
-                                  int h_dtype, int w_dtype, void* stream) {
+B200_API int b200_sandwich_norm_2(const void* y, const void* w_post, const void* y2, const void* w_post2, const float* res_in,
+                                  float* res_out, const void* w_next, void* h, long long rows, int cols, float eps, float off,
+                                  float mult, int center, int y_dtype, int h_dtype, int w_dtype, void* stream) {
   using namespace b200;
   cudaStream_t st = (cudaStream_t)stream;
   if (rows <= 0) return 0;
-  if (cols <= 0) return B200_ERR_BAD_SHAPE;
+  if (cols <= 0 || (y2 && (!y || !w_post || !w_post2 || center))) return B200_ERR_BAD_SHAPE;
   typedef __nv_bfloat16 bf;
-#define SW(TY, TH, WT) return sandwich_launch<TY, TH, WT>(y, w_post, res_in, res_out, w_next, h, rows, cols, eps, off, mult, center, st)
+#define SW(TY, TH, WT) return sandwich_launch<TY, TH, WT>(y, w_post, y2, w_post2, res_in, res_out, w_next, h, rows, cols, eps, off, mult, center, st)
   if (w_dtype == B200_DT_BF16) {
     if (y_dtype == B200_DT_FP32 && h_dtype == B200_DT_BF16) SW(float, bf, bf);
     if (y_dtype == B200_DT_BF16 && h_dtype == B200_DT_BF16) SW(bf, bf, bf);
@@ -562,6 +576,13 @@ B200_API int b200_sandwich_norm_c(const void* y, const void* w_post, const float
   }
 #undef SW
   return B200_ERR_UNSUPPORTED;
+}
+
+B200_API int b200_sandwich_norm_c(const void* y, const void* w_post, const float* res_in, float* res_out, const void* w_next,
+                                  void* h, long long rows, int cols, float eps, float off, float mult, int center, int y_dtype,
+                                  int h_dtype, int w_dtype, void* stream) {
+  return b200_sandwich_norm_2(y, w_post, nullptr, nullptr, res_in, res_out, w_next, h, rows, cols, eps, off, mult, center, y_dtype, h_dtype,
+                              w_dtype, stream);
 }
 
 B200_API int b200_sandwich_norm(const void* y, const void* w_post, const float* res_in, float* res_out, const void* w_next,

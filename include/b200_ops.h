@@ -415,6 +415,10 @@ int b200_flash_attn_bwd_tc(const void* qkv, const void* out, const void* dout, c
  * LLM_on_Kubernetes/Inference_Platfrom/README.md:1504-1511). */
 int b200_gemv16(const void* x, const void* w, const void* bias, void* y, int M, long long N, int K, long long x_rs,
                 long long w_rs, long long y_rs, int dtype, int out_f32, void* stream);
+/* The same for `batch` problems in one launch, operands x_bs / w_bs / y_bs elements apart. */
+int b200_gemv16_batched(const void* x, const void* w, const void* bias, void* y, int M, long long N, int K, long long x_rs,
+                        long long w_rs, long long y_rs, int batch, long long x_bs, long long w_bs, long long y_bs, int dtype,
+                        int out_f32, void* stream);
 int b200_w4_gemv_batched(const void* x, const uint8_t* packed, const float* scale, const float* zs, const float* lut,
                          const void* bias, void* y, int M, long long N, int K, int group, long long x_rs, long long y_rs,
                          int dtype, void* stream);
@@ -476,6 +480,10 @@ int b200_paged_attn_mma(const void* q, long long q_stride, const void* ck, const
 int b200_sandwich_norm(const void* y, const void* w_post, const float* res_in, float* res_out, const void* w_next, void* h,
                        long long rows, int cols, float eps, float off, float mult, int y_dtype, int h_dtype, int w_dtype,
                        void* stream);
+/* The same with a second branch y2 (NULL: none): x = res_in + mult * (rms(y) * (off + w_post) + rms(y2) * (off + w_post2)); center 0. */
+int b200_sandwich_norm_2(const void* y, const void* w_post, const void* y2, const void* w_post2, const float* res_in, float* res_out,
+                         const void* w_next, void* h, long long rows, int cols, float eps, float off, float mult, int center,
+                         int y_dtype, int h_dtype, int w_dtype, void* stream);
 /* The same with `center` 1: both norms are layer norms without a bias ((x - mean) / sqrt(variance + eps) * (off + w)). */
 int b200_sandwich_norm_c(const void* y, const void* w_post, const float* res_in, float* res_out, const void* w_next, void* h,
                          long long rows, int cols, float eps, float off, float mult, int center, int y_dtype, int h_dtype,
@@ -537,6 +545,8 @@ int b200_latent_attn_mma(const void* q, const void* cache, const int* tiles, int
                          const int* table, int max_blocks, const float* sinks, void* out, float* part, int H, int Dk, int Dv,
                          int block_size, float scale, int nsplit, int dtype, void* stream);
 /* D [M, N] = A [M, K] B[N, K]^T in true fp32 (FFMA; no TF32 rounding of the operands); any sizes and row strides. */
+int b200_gemm_f32_exact_bias(const float* A, const float* B, const float* bias, float* D, int M, int N, int K, long long lda,
+                             long long ldb, long long ldd, void* stream);      /* bias fp32 [N] or NULL */
 int b200_gemm_f32_exact(const float* A, const float* B, float* D, int M, int N, int K, long long lda, long long ldb, long long ldd,
                         void* stream);
 
@@ -564,6 +574,21 @@ int b200_qknorm_rope_store(const float* proj, long long ld, const float* wq, con
                            const float* sin_t, const int* pos, const int* slot, const int* table, int max_blocks, void* q_out,
                            void* ck, void* cv, int tokens, int H, int G, int M, int D, int Dv, int rot, int block_size, float eps,
                            int has_kv, int dtype, void* stream);
+/* The same with every part optional: bias fp32 per column of proj or NULL; wq / wk NULL: rows are not normed; rot 0: no rotation;
+ * v_first (a pool shaped like cv, filled for these tokens) with v_lambda fp32 [1]: v <- (1 - lambda) v + lambda v_first.
+ * proj in x_dtype (fp32, or bf16 with a bf16 cache); D and Dv <= 512. */
+int b200_qkv_store(const void* proj, long long ld, const float* bias, const float* wq, const float* wk, const float* cos_t,
+                   const float* sin_t, const int* pos, const int* slot, const int* table, int max_blocks, void* q_out, void* ck,
+                   void* cv, const void* v_first, const float* v_lambda, int tokens, int H, int G, int M, int D, int Dv, int rot,
+                   int block_size, float eps, int has_kv, int x_dtype, int dtype, void* stream);
+/* Options of one-map attention; a zeroed struct is none of them. */
+typedef struct b200_attn_opts {
+  const float* sink;       /* [H]: exp(sink_h) joins the softmax's denominator (no key, no value, not scaled) */
+  const float* gate;       /* [tokens] rows of stride ld_gate holding H: o_h is multiplied by sigmoid(gate_h) */
+  long long ld_gate;
+  float softcap;           /* > 0: scores become cap tanh(s / cap) */
+  int chunk;               /* > 0: token at p sees only keys j with j / chunk == p / chunk (window must be <= 0) */
+} b200_attn_opts;
 /* out, rows of stride ldo holding H * Dv: token t sees key j <= pos[t] of its row if pos[t] - j < window or j < keep_first (window <= 0: all).
  * Each of the M maps is a softmax attention over the same values; combine (M = 2): o = a_0 - lambda a_1, then
  * o / sqrt(mean(o^2) + eps); the result is multiplied by post. Dv <= 256. fp32 arithmetic. nsplit > 1 cuts every token's visible keys into ranges
@@ -572,9 +597,18 @@ int b200_multimap_attn(const void* q, const void* ck, const void* cv, const int*
                        int max_blocks, void* out, long long ldo, float* part, int tokens, int H, int G, int M, int D, int Dv, int block_size,
                        float scale, int window, int keep_first, int nsplit, int combine, float lambda, float post, float eps,
                        int dtype, void* stream);
+/* The same with options (opts may be NULL; M = 1 otherwise). */
+int b200_multimap_attn_ex(const void* q, const void* ck, const void* cv, const int* pos, const int* slot, const int* table,
+                          int max_blocks, void* out, long long ldo, float* part, int tokens, int H, int G, int M, int D, int Dv, int block_size,
+                          float scale, int window, int keep_first, int nsplit, int combine, float lambda, float post, float eps,
+                          const b200_attn_opts* opts, int dtype, void* stream);
+int b200_multimap_attn_mma_ex(const void* q, const void* ck, const void* cv, const int* tiles, int n_tiles, const int* table,
+                              int max_blocks, void* out, long long ldo, int H, int G, int M, int D, int Dv, int block_size, float scale,
+                              int window, int keep_first, int combine, float lambda, float post, float eps, const b200_attn_opts* opts,
+                              int dtype, void* stream);
 /* The same for bf16 prompt pieces on mma.sync: tiles int32 [n_tiles, 4] = (first row, rows <= 64, position of the first row,
- * cache row). D in {32, 48, 64, 96, 128}, Dv in {32, 64, 96, 128}, block_size a power of two, scale > 0; else
- * B200_ERR_UNSUPPORTED (use b200_multimap_attn). */
+ * cache row). D and Dv multiples of 8 up to 128, block_size a power of two, scale > 0; else B200_ERR_UNSUPPORTED (use
+ * b200_multimap_attn). */
 int b200_multimap_attn_mma(const void* q, const void* ck, const void* cv, const int* tiles, int n_tiles, const int* table,
                            int max_blocks, void* out, long long ldo, int H, int G, int M, int D, int Dv, int block_size, float scale, int window,
                            int keep_first, int combine, float lambda, float post, float eps, int dtype, void* stream);
@@ -609,11 +643,20 @@ int b200_short_conv_ex(const void* x, long long ldx, const float* w, const float
 int b200_silu_rows(float* x, long long ld, long long rows, int cols, void* stream);
 int b200_short_conv_tail(const void* x, long long ldx, const float* in_bias, float* state, const int* runs, const int* pos,
                          const int* slot, int n_runs, int C, int taps, int x_dtype, void* stream);
+/* b200_delta_gates with AD decays per head: a [tokens, H * AD], dt_bias [H * AD], AD = D or 1. */
+int b200_delta_gates_ex(float* q, long long ldq, float* k, long long ldk, float* a, long long lda, float* b, long long ldb,
+                        const float* dt_bias, const float* A_log, int tokens, int G, int H, int D, int AD, float qscale,
+                        float unit_eps, void* stream);
+/* out[s, t] = h[t] + (h' - h[t]) mu[s] for the S rows of mu (fp32 [S, W]); h' is the row before in the token's run, at the start of
+ * a run the row of prev (fp32 [rows, W]), at position 0 zero. step_tail 1: every token is a run of its own and prev is replaced
+ * in the same launch; else b200_short_conv_tail (two taps) advances it. h [tokens, W] and out [S, tokens, W] in dtype (fp32 / bf16). */
+int b200_token_shift(const void* h, long long ldh, const float* mu, float* prev, const int* pos, const int* slot, void* out,
+                     int tokens, int W, int S, int step_tail, int dtype, void* stream);
 int b200_delta_gates(float* q, long long ldq, float* k, long long ldk, float* a, long long lda, float* b, long long ldb,
                      const float* dt_bias, const float* A_log, int tokens, int G, int H, int D, float qscale, float unit_eps,
                      void* stream);
 /* mode 0: S <- decay[h] S + k v^T; mode 1: S <- diag(g) S, u = beta (v - S^T k), S <- S + k u^T; mode 2: S <- a S + b k v^T
- * with one a and b per token and head (g = a [tokens, H], beta = b [tokens, H]); o = S^T q (fp32 [tokens, H, Dv]). q / k have G
+ * with one a and b per token and head (g = a [tokens, H], beta = b [tokens, H]); mode 3: mode 1 with one decay per token and head (g [tokens, H]); o = S^T q (fp32 [tokens, H, Dv]). q / k have G
  * heads of D (head h reads h / (H / G)), v H heads of Dv - ones, g [tokens, H * D] in mode 1, beta [tokens, H]. act 1: silu on q,
  * k, v as they are read. ones 1: a column of ones is appended to every head of v (Dv counts it). state fp32 [rows, H, D, Dv]. */
 int b200_linear_scan(const float* q, long long ldq, const float* k, long long ldk, const float* v, long long ldv, const float* g,
@@ -630,20 +673,23 @@ int b200_ssm_gates(const float* dt, long long ld, const float* dt_bias, const fl
                    int H, void* stream);
 /* Per token: v = o[h, d] * oscale; e != NULL: v /= max(|o[h, Dv] * oscale|, e[t, h]) + den_eps; skip != NULL: v += skip[h] x[c];
  * pre != NULL: v *= silu(pre[c]); RMS norm over `groups` equal column groups; times w (w_full 1: [H * Dv], 0: [group size]);
- * post != NULL: v *= sigmoid(post[c]), or silu(post[c]) with post_silu 1. o fp32 [tokens, H, ocols]; out [tokens, H * Dv] in out_dtype. */
+ * post != NULL: v *= sigmoid(post[c]), or silu(post[c]) with post_silu 1 (post in post_dtype: fp32, or bf16 with a bf16 out). o fp32 [tokens, H, ocols]; out [tokens, H * Dv] in out_dtype. */
 int b200_scan_readout(const float* o, int ocols, const float* e, float den_eps, float oscale, const float* skip, const float* x,
-                      long long ldx, const float* pre, long long ldpre, const float* post, long long ldpost, int post_silu,
-                      const float* w, int w_full, void* out, long long tokens, int H, int Dv, int groups, float eps, int out_dtype, void* stream);
+                      long long ldx, const float* pre, long long ldpre, const void* post, long long ldpost, int post_silu,
+                      int post_dtype, const float* w, int w_full, void* out, long long tokens, int H, int Dv, int groups, float eps, int out_dtype, void* stream);
 
 /* Per-channel decays of a low-rank input and the scan that uses them (csrc/channel_scan.cu): out[t, c] = sigmoid(w2[c] . x[t] +
- * bias[c])^inv_tau (fast 1: hardware exponential and logarithm); per head S <- diag(g) S + k v^T, o = S^T q (fp32). n_tiles > 0: runs are walked tile by tile in parallel,
+ * bias[c])^inv_tau (fast 1: hardware exponential and logarithm), _ex with form 1: exp(-exp(w2[c] . tanh(x[t]) + bias[c])); per head
+ * S <- diag(g) S + k v^T, o = S^T q, or with u (fp32 [H, D]) o = (S + diag(u) k v^T)^T q before that update (fp32). n_tiles > 0: runs are walked tile by tile in parallel,
  * tiles int32 [n_tiles, 4] = (first row, rows, first position, state row), tile_of [n_tiles, 4] = (run, place in the run, tiles
  * of the run, its first tile), run_tiles [n_runs, 4] = (first tile, tiles, 0, 0), part fp32 [n_tiles, H, D, Dv] and pdec fp32
  * [n_tiles, H, D] are scratch. chunk: tokens staged at a time (at most 16). */
 int b200_lowrank_decay(const float* x, long long ldx, const float* w2, const float* bias, float* out, int tokens, int C, int rank,
                        float inv_tau, int fast, void* stream);
+int b200_lowrank_decay_ex(const float* x, long long ldx, const float* w2, const float* bias, float* out, int tokens, int C, int rank,
+                          float inv_tau, int form, int fast, void* stream);
 int b200_channel_scan(const float* q, long long ldq, const float* k, long long ldk, const float* v, long long ldv, const float* g,
-                      long long ldg, float* state, float* part, float* pdec, const int* runs, int n_runs, const int* tiles,
+                      long long ldg, const float* u, float* state, float* part, float* pdec, const int* runs, int n_runs, const int* tiles,
                       int n_tiles, const int* tile_of, const int* run_tiles, int chunk, const int* pos, const int* slot, float* o,
                       int H, int G, int D, int Dv, void* stream);
 /* Selective state space with a decay per channel and state (csrc/selective_scan.cu): s = softplus(dt + dt_bias), S[n, c] <-

@@ -31,6 +31,11 @@ def _load_lorenex(path, dtype, device):
     return lorenex_from_pretrained(path, dtype=dtype, device=device)
 
 
+def _load_nedesun(path, dtype, device):
+    from .nedesun import nedesun_from_pretrained
+    return nedesun_from_pretrained(path, dtype=dtype, device=device)
+
+
 # ``architecture`` (or HF ``model_type`` / ``architectures[0]``) of config.json -> loader(path, dtype, device).
 # Anything not listed is read as a Qwen2/Qwen3-style HF checkpoint by ``io.hf.from_pretrained``.
 MODEL_REGISTRY: Dict[str, Callable] = {
@@ -44,6 +49,8 @@ MODEL_REGISTRY: Dict[str, Callable] = {
     "kudonex": _load_kudonex,
     "Lorenex": _load_lorenex,
     "lorenex": _load_lorenex,
+    "Nedesun": _load_nedesun,
+    "nedesun": _load_nedesun,
 }
 
 

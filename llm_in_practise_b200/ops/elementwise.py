@@ -347,9 +347,10 @@ def sinusoid_table(n: int, width: int, device, base: float = 10000.0) -> torch.T
     return tab.to(torch.float32).contiguous().to(device)
 
 
-def embedding_pos(ids: torch.Tensor, table: torch.Tensor, scale: float, pos: torch.Tensor, pos_table: torch.Tensor) -> torch.Tensor:
+def embedding_pos(ids: torch.Tensor, table: torch.Tensor, scale: float, pos: Optional[torch.Tensor] = None,
+                  pos_table: Optional[torch.Tensor] = None) -> torch.Tensor:
     """fp32 [T, W] = ``table[ids] * scale + pos_table[pos]``: embedding rows entering an fp32 stream, every token with its own
-    position (``pos`` int32 [T], ``pos_table`` fp32 [positions, W])."""
+    position (``pos`` int32 [T], ``pos_table`` fp32 [positions, W]; None: nothing is added)."""
     T, W = ids.shape[0], table.shape[1]
     if nv.use_native(table):
         out = torch.empty(T, W, dtype=torch.float32, device=table.device)
@@ -358,7 +359,8 @@ def embedding_pos(ids: torch.Tensor, table: torch.Tensor, scale: float, pos: tor
                     nv.dtype_code(table.dtype), nv.stream()), "embedding_pos")
         nv.count_launch()
         return out
-    return table[ids].float() * scale + pos_table[pos.long()]
+    x = table[ids].float() * scale
+    return x if pos_table is None else x + pos_table[pos.long()]
 
 
 # ------------------------------------------------------------------------------------------------

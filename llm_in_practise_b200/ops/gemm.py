@@ -334,22 +334,24 @@ def gemm_w4(a: torch.Tensor, q, *, b_mn: bool = False, out: Optional[torch.Tenso
     return out
 
 
-def linear_exact(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
-    """``x @ w^T`` for inference at the precision of the operands: 16-bit operands go to the tcgen05 GEMM (fp32
+def linear_exact(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
+                 bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``x @ w^T`` (+ ``bias`` [N], in x's dtype) for inference at the precision of the operands: 16-bit operands go to the tcgen05 GEMM (fp32
     accumulation, ``out_dtype`` output), fp32 operands to the FFMA kernel ``b200_gemm_f32_exact`` — the tensor-core route
     would round them to TF32, which a run that asks for fp32 must not do. Operand rows whose byte stride is not a multiple
     of 16 (K % 8 for 16-bit) cannot be described to TMA; they are multiplied in fp32 by the same FFMA kernel."""
     out_dtype = out_dtype or x.dtype
     if not nv.use_native(x):
-        return (x.float() @ w.float().t()).to(out_dtype)
+        y = x.float() @ w.float().t()
+        return (y if bias is None else y + bias.float()).to(out_dtype)
     M, K = x.shape
     N = w.shape[0]
     if x.dtype != torch.float32 and K % 8 == 0:
         if M <= 16 and out_dtype in (x.dtype, torch.float32):
-            y = gemv16(x, w, out_dtype=out_dtype)
+            y = gemv16(x, w, bias=bias, out_dtype=out_dtype)
             if y is not None:
                 return y
-        return gemm(x, w, out_dtype=out_dtype)
+        return gemm(x, w, bias=bias, out_dtype=out_dtype)
     xf = x if x.dtype == torch.float32 else x.float()
     wf = w if w.dtype == torch.float32 else w.float()
     if xf.stride(-1) != 1:
@@ -358,10 +360,33 @@ def linear_exact(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dty
         wf = wf.contiguous()
     y = torch.empty(M, N, dtype=torch.float32, device=x.device)
     vp, i32, i64 = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong
-    fn = nv.proto("b200_gemm_f32_exact", [vp, vp, vp, i32, i32, i32, i64, i64, i64, vp])
-    nv.check(fn(nv.ptr(xf), nv.ptr(wf), nv.ptr(y), M, N, K, xf.stride(0), wf.stride(0), y.stride(0), nv.stream()), "gemm_f32_exact")
+    fn = nv.proto("b200_gemm_f32_exact_bias", [vp, vp, vp, vp, i32, i32, i32, i64, i64, i64, vp])
+    bf = bias.float() if bias is not None else None
+    nv.check(fn(nv.ptr(xf), nv.ptr(wf), nv.ptr(bf), nv.ptr(y), M, N, K, xf.stride(0), wf.stride(0), y.stride(0), nv.stream()), "gemm_f32_exact")
     nv.count_launch()
     return y if out_dtype == torch.float32 else y.to(out_dtype)
+
+
+def linear_each(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """Several projections of equal size, each of an input of its own: ``x`` [B, M, K], ``w`` [B, N, K] -> fp32 [M, B * N], product
+    b in columns b N .. (b + 1) N, at the precision of the operands (see ``linear_exact``). 16-bit operands are one launch: the
+    small-M kernel with a batch dimension, or the batched tcgen05 GEMM."""
+    B, M, K = x.shape
+    N = w.shape[1]
+    out = torch.empty(M, B, N, dtype=torch.float32, device=x.device)
+    if nv.use_native(x) and x.dtype != torch.float32 and K % 8 == 0 and N % 8 == 0 and x.is_contiguous() and w.is_contiguous():
+        if M <= 16 and K % 128 == 0 and w.dtype == x.dtype and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0:
+            vp, i32, i64 = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong
+            fn = nv.proto("b200_gemv16_batched", [vp, vp, vp, vp, i32, i64, i32, i64, i64, i64, i32, i64, i64, i64, i32, i32, vp])
+            nv.check(fn(nv.ptr(x), nv.ptr(w), None, nv.ptr(out), M, N, K, K, K, B * N, B, M * K, N * K, N, nv.dtype_code(x.dtype), 1,
+                        nv.stream()), f"gemv16_batched M={M} N={N} K={K} B={B}")
+            nv.count_launch()
+        else:
+            gemm(x, w, out=out.transpose(0, 1))
+    else:
+        for b in range(B):
+            out[:, b] = linear_exact(x[b], w[b], out_dtype=torch.float32)
+    return out.view(M, B * N)
 
 
 def head_linear(x: torch.Tensor, w: torch.Tensor, w_kn: bool = False, out: Optional[torch.Tensor] = None) -> torch.Tensor:

@@ -9,12 +9,15 @@ run that starts at position 0 starts from a zero state, so state rows are reused
 
     silu_rows_     x <- silu(x) on a column slice of fp32 rows
     short_conv     y[t, c] = act(sum_j w[c, j] x[t - (taps - 1) + j, c]); the tail [rows, taps - 1, C] holds the last inputs
-    delta_gates    unit q / k per head, decays exp(-exp(A_log) softplus(a + bias)), beta = sigmoid(b), in place
+    token_shift    h + (h' - h) mu_s for several mu_s, h' the previous token's h (carried in a state row)
+    delta_gates    unit q / k per head, decays exp(-exp(A_log) softplus(a + bias)) per key channel or per head, beta = sigmoid(b), in place
     linear_scan    mode "decay":  S <- decay_h S + k v^T;                                  o = S^T q
                    mode "delta":  S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T;    o = S^T q
                    mode "gated":  S <- a_t S + b_t k v^T (one a, b per token and head);    o = S^T q
-                   mode "channel": S <- diag(g) S + k v^T (a decay per key channel);       o = S^T q
-    lowrank_decay  per-channel decays sigmoid(W_2 x + bias)^(1 / tau) of a low-rank input x
+                   mode "channel": S <- diag(g) S + k v^T (a decay per key channel);       o = S^T q, or with a bonus u for
+                                   the current token o = (S + diag(u) k v^T)^T q, read before the update
+                   mode "head_delta": "delta" with one decay per token and head
+    lowrank_decay  per-channel decays sigmoid(W_2 x + bias)^(1 / tau), or exp(-exp(W_2 tanh(x) + bias)), of a low-rank input x
     selective_scan S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c u_c B_n; y_c = sum_n S[c, n] C_n + D_c u_c; y silu(gate) scale
     mlstm_gates    capped log gates of an mLSTM and their running maximum -> (a, b, exp(-m)) for the gated scan
     ssm_gates      dt = softplus(x + bias), a = exp(-exp(A_log) dt), b = dt: the step sizes of a selective state space
@@ -87,6 +90,34 @@ def _conv_tail(x, in_bias, tail, runs, pos, slot, n_runs, C, taps):
     nv.count_launch()
 
 
+def token_shift(h: torch.Tensor, mu: torch.Tensor, prev: torch.Tensor, pos: torch.Tensor, slot: torch.Tensor,
+                runs: Optional[torch.Tensor], n_runs: int) -> torch.Tensor:
+    """``h`` [T, W], ``mu`` fp32 [S, W] -> [S, T, W] in h's dtype: row s is ``h + (h' - h) mu[s]`` with h' the h of the token before
+    (zeros at position 0). ``prev`` fp32 [rows, 1, W] holds the last token's h of every sequence and is advanced over the runs
+    (one launch for a decode batch, two otherwise)."""
+    T, W = h.shape
+    S = mu.shape[0]
+    if nv.use_native(h):
+        if h.dtype not in (torch.float32, torch.bfloat16) or h.stride(1) != 1:
+            raise ValueError("token_shift: fp32 or bf16 rows with a contiguous last dim")
+        out = torch.empty(S, T, W, dtype=h.dtype, device=h.device)
+        fn = nv.proto("b200_token_shift", [vp, i64, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, vp])
+        nv.check(fn(nv.ptr(h), h.stride(0), nv.ptr(mu), nv.ptr(prev), nv.ptr(pos), nv.ptr(slot), nv.ptr(out), T, W, S, int(runs is None),
+                    nv.dtype_code(h.dtype), nv.stream()), "token_shift")
+        nv.count_launch()
+        if runs is not None:
+            _conv_tail(h, None, prev, runs, pos, slot, n_runs, W, 2)
+        return out
+    before = torch.zeros(T, W, dtype=torch.float32, device=h.device)
+    for first, n, p0, s in _run_list(runs, pos, slot):
+        if p0 > 0:
+            before[first] = prev[s, 0]
+        before[first + 1:first + n] = h[first:first + n - 1].float()
+        prev[s, 0] = h[first + n - 1].float()
+    hf = h.float()
+    return torch.stack([hf + (before - hf) * mu[i].float() for i in range(S)]).to(h.dtype)
+
+
 def silu_rows_(x: torch.Tensor) -> torch.Tensor:
     """In place ``silu`` on an fp32 [T, C] view whose rows may be strided (a column slice of a fused projection)."""
     if nv.use_native(x):
@@ -103,42 +134,48 @@ def silu_rows_(x: torch.Tensor) -> torch.Tensor:
 def delta_gates(q: torch.Tensor, k: torch.Tensor, a: torch.Tensor, b: torch.Tensor, dt_bias: torch.Tensor, A_log: torch.Tensor,
                 G: int, H: int, D: int, qscale: float, unit_eps: float = 1e-6) -> None:
     """In place on fp32 views with strided rows: q, k [T, G * D] -> x / sqrt(sum(x^2) + unit_eps) per head (q also times
-    ``qscale``); a [T, H * D] -> exp(-exp(A_log[h]) * softplus(a + dt_bias)); b [T, H] -> sigmoid(b)."""
+    ``qscale``); a [T, H * D] (a decay per key channel) or [T, H] (one per head) -> exp(-exp(A_log[h]) * softplus(a + dt_bias));
+    b [T, H] -> sigmoid(b)."""
     T = q.shape[0]
+    AD = a.shape[1] // H
     if nv.use_native(q):
-        fn = nv.proto("b200_delta_gates", [vp, i64, vp, i64, vp, i64, vp, i64, vp, vp, i32, i32, i32, i32, f32, f32, vp])
+        fn = nv.proto("b200_delta_gates_ex", [vp, i64, vp, i64, vp, i64, vp, i64, vp, vp, i32, i32, i32, i32, i32, f32, f32, vp])
         nv.check(fn(nv.ptr(q), q.stride(0), nv.ptr(k), k.stride(0), nv.ptr(a), a.stride(0), nv.ptr(b), b.stride(0), nv.ptr(dt_bias),
-                    nv.ptr(A_log), T, G, H, D, float(qscale), float(unit_eps), nv.stream()), "delta_gates")
+                    nv.ptr(A_log), T, G, H, D, AD, float(qscale), float(unit_eps), nv.stream()), "delta_gates")
         nv.count_launch()
         return
     for x, sc in ((q, qscale), (k, 1.0)):
         v = x.view(T, G, D)
         x.copy_((v * torch.rsqrt((v * v).sum(-1, keepdim=True) + unit_eps) * sc).view(T, G * D))
-    a.copy_(torch.exp(-torch.exp(A_log.float()).view(1, H, 1) * F.softplus(a.view(T, H, D) + dt_bias.float().view(1, H, D))).view(T, H * D))
+    a.copy_(torch.exp(-torch.exp(A_log.float()).view(1, H, 1) * F.softplus(a.reshape(T, H, AD) + dt_bias.float().view(1, H, AD))).view(T, H * AD))
     b.copy_(torch.sigmoid(b))
 
 
-SCAN_MODES = ("decay", "delta", "gated", "channel")
+SCAN_MODES = ("decay", "delta", "gated", "channel", "head_delta")
+_KERNEL_MODE = {"decay": 0, "delta": 1, "gated": 2, "head_delta": 3}
 
 
 def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, pos: torch.Tensor, slot: torch.Tensor,
                 runs: Optional[torch.Tensor], n_runs: int, H: int, G: int, D: int, Dv: int, mode: str,
                 decay: Optional[torch.Tensor] = None, g: Optional[torch.Tensor] = None, beta: Optional[torch.Tensor] = None,
-                act: bool = False, ones: bool = False, pieces=None) -> torch.Tensor:
+                act: bool = False, ones: bool = False, pieces=None, u: Optional[torch.Tensor] = None) -> torch.Tensor:
     """o fp32 [T, H * Dv]. q, k fp32 [T, G * D] (head h reads head h // (H / G)), v fp32 [T, H * Dv] (rows may be strided);
     ``state`` fp32 [rows, H, D, Dv] is read at the start of each run and written at its end. ``mode`` "decay" takes
     ``decay`` fp32 [H]; "delta" takes ``g`` fp32 [T, H * D] (per key channel) and ``beta`` fp32 [T, H]; "gated" takes
-    ``g`` = a and ``beta`` = b, both fp32 [T, H]; "channel" takes ``g`` fp32 [T, H * D] alone. ``act``: silu on q, k and v as they are read. ``ones``: every head of v gets
+    ``g`` = a and ``beta`` = b, both fp32 [T, H], and so does "head_delta" its decay and beta; "channel" takes ``g`` fp32
+    [T, H * D] and optionally the bonus ``u`` fp32 [H, D]. ``act``: silu on q, k and v as they are read. ``ones``: every head of v gets
     one more column, all ones — ``Dv`` counts it, v itself has ``Dv - 1`` columns per head — so the state's last column
     accumulates the decayed b k alone and o's last column is its product with q. ``pieces`` (``inference.ragged.Pieces``,
     mode "channel"): runs of several tiles are walked tile by tile in parallel, see ``csrc/linear_scan.cu``."""
     T = q.shape[0]
     o = torch.empty(T, H * Dv, dtype=torch.float32, device=q.device)
-    delta = mode == "delta"
+    delta = mode in ("delta", "head_delta")
     gated = mode == "gated"
     channel = mode == "channel"
     if mode not in SCAN_MODES:
         raise ValueError(f"linear_scan: no mode {mode!r}")
+    if u is not None and not channel:
+        raise ValueError("linear_scan: a bonus goes with mode \"channel\"")
     if nv.use_native(q) and channel:
         if act or ones:
             raise ValueError("linear_scan: mode \"channel\" takes neither act nor ones")
@@ -148,10 +185,10 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.
         pdec = torch.empty(nt * H * D, dtype=torch.float32, device=q.device) if tiled else None
         longest = 1 if runs is None else (pieces.longest if pieces is not None else 16)
         opt = lambda name: nv.ptr(getattr(pieces, name) if tiled else None)                      # noqa: E731
-        fn = nv.proto("b200_channel_scan", [vp, i64, vp, i64, vp, i64, vp, i64, vp, vp, vp, vp, i32, vp, i32, vp, vp, i32, vp, vp, vp,
+        fn = nv.proto("b200_channel_scan", [vp, i64, vp, i64, vp, i64, vp, i64, vp, vp, vp, vp, vp, i32, vp, i32, vp, vp, i32, vp, vp, vp,
                                             i32, i32, i32, i32, vp])
-        nv.check(fn(nv.ptr(q), q.stride(0), nv.ptr(k), k.stride(0), nv.ptr(v), v.stride(0), nv.ptr(g), g.stride(0), nv.ptr(state),
-                    nv.ptr(part), nv.ptr(pdec), nv.ptr(runs), n_runs if runs is not None else T, opt("tiles"), nt, opt("tile_of"),
+        nv.check(fn(nv.ptr(q), q.stride(0), nv.ptr(k), k.stride(0), nv.ptr(v), v.stride(0), nv.ptr(g), g.stride(0), nv.ptr(u),
+                    nv.ptr(state), nv.ptr(part), nv.ptr(pdec), nv.ptr(runs), n_runs if runs is not None else T, opt("tiles"), nt, opt("tile_of"),
                     opt("run_tiles"), longest, nv.ptr(pos), nv.ptr(slot), nv.ptr(o), H, G, D, Dv, nv.stream()), "channel_scan")
         nv.count_launch(3 if tiled else 1)
         return o
@@ -161,7 +198,7 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.
         per = delta or gated
         nv.check(fn(nv.ptr(q), q.stride(0), nv.ptr(k), k.stride(0), nv.ptr(v), v.stride(0), nv.ptr(g), g.stride(0) if per else 0,
                     nv.ptr(beta), beta.stride(0) if beta is not None else 0, nv.ptr(decay), nv.ptr(state), nv.ptr(runs), nv.ptr(pos),
-                    nv.ptr(slot), n_runs if runs is not None else T, nv.ptr(o), H, G, D, Dv, SCAN_MODES.index(mode), int(act),
+                    nv.ptr(slot), n_runs if runs is not None else T, nv.ptr(o), H, G, D, Dv, _KERNEL_MODE[mode], int(act),
                     int(ones), nv.stream()), "linear_scan")
         nv.count_launch()
         return o
@@ -177,12 +214,17 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.
         S = state[s].clone() if p0 > 0 else torch.zeros(H, D, Dv, dtype=torch.float32, device=q.device)
         for t in range(first, first + n):
             if delta:
-                S = S * g[t].view(H, D, 1)
-                u = beta[t].view(H, 1) * (vf[t] - torch.einsum("hde,hd->he", S, kf[t]))
-                S = S + kf[t][:, :, None] * u[:, None, :]
+                S = S * g[t].reshape(H, -1, 1)
+                w = beta[t].reshape(H, 1) * (vf[t] - torch.einsum("hde,hd->he", S, kf[t]))
+                S = S + kf[t][:, :, None] * w[:, None, :]
             elif gated:
                 S = g[t].float().view(H, 1, 1) * S + kf[t][:, :, None] * (beta[t].float().view(H, 1) * vf[t])[:, None, :]
             elif channel:
+                if u is not None:
+                    kv = kf[t][:, :, None] * vf[t][:, None, :]
+                    ov[t] = torch.einsum("hde,hd->he", S + u.float().view(H, D, 1) * kv, qf[t])
+                    S = S * g[t].float().reshape(H, D, 1) + kv
+                    continue
                 S = S * g[t].float().reshape(H, D, 1) + kf[t][:, :, None] * vf[t][:, None, :]
             else:
                 S = decay.float().view(H, 1, 1) * S + kf[t][:, :, None] * vf[t][:, None, :]
@@ -243,18 +285,18 @@ def scan_readout(o: torch.Tensor, H: int, Dv: int, w: torch.Tensor, groups: int,
     a column of ones (``e`` fp32 [T, H] given: v = oscale o[h, :Dv] / (max(|oscale o[h, Dv]|, e[h]) + den_eps)); ``skip`` fp32
     [H] with ``x`` fp32 [T, H * Dv]: v += skip[h] x; ``pre``: v *= silu(pre); RMS norm over ``groups`` equal parts of the
     H * Dv columns; times ``w`` (fp32, one per column, or one per column of a group); ``post``: v *= sigmoid(post), or silu(post) with ``post_act`` "silu". pre / post /
-    x are fp32 rows that may be strided. Returns [T, H * Dv] in ``out_dtype``."""
+    x are fp32 rows that may be strided (post may be bf16 when the output is). Returns [T, H * Dv] in ``out_dtype``."""
     T = o.shape[0]
     N = H * Dv
     ocols = o.shape[1] // H
     w_full = w.numel() == N
     if nv.use_native(o):
         out = torch.empty(T, N, dtype=out_dtype, device=o.device)
-        fn = nv.proto("b200_scan_readout", [vp, i32, vp, f32, f32, vp, vp, i64, vp, i64, vp, i64, i32, vp, i32, vp, i64, i32, i32, i32,
-                                            f32, i32, vp])
+        fn = nv.proto("b200_scan_readout", [vp, i32, vp, f32, f32, vp, vp, i64, vp, i64, vp, i64, i32, i32, vp, i32, vp, i64, i32, i32,
+                                            i32, f32, i32, vp])
         st = lambda z: z.stride(0) if z is not None else 0                      # noqa: E731
         nv.check(fn(nv.ptr(o), ocols, nv.ptr(e), float(den_eps), float(oscale), nv.ptr(skip), nv.ptr(x), st(x), nv.ptr(pre), st(pre),
-                    nv.ptr(post), st(post), int(post_act == "silu"), nv.ptr(w), int(w_full), nv.ptr(out), T, H, Dv, groups, float(eps),
+                    nv.ptr(post), st(post), int(post_act == "silu"), nv.dtype_code(post.dtype if post is not None else torch.float32), nv.ptr(w), int(w_full), nv.ptr(out), T, H, Dv, groups, float(eps),
                     nv.dtype_code(out_dtype), nv.stream()), "scan_readout")
         nv.count_launch()
         return out
@@ -275,19 +317,23 @@ def scan_readout(o: torch.Tensor, H: int, Dv: int, w: torch.Tensor, groups: int,
     return v.to(out_dtype)
 
 
-def lowrank_decay(x: torch.Tensor, w2: torch.Tensor, bias: torch.Tensor, tau: float, fast: bool = False) -> torch.Tensor:
-    """``x`` fp32 [T, r] (rows may be strided), ``w2`` fp32 [C, r], ``bias`` fp32 [C] -> sigmoid(w2 x + bias)^(1 / tau), fp32
-    [T, C], formed as exp(log sigmoid(.) / tau). ``fast``: with the hardware's exponential and logarithm (models in 16 bits)."""
+def lowrank_decay(x: torch.Tensor, w2: torch.Tensor, bias: torch.Tensor, tau: float = 1.0, fast: bool = False,
+                  form: str = "sigmoid") -> torch.Tensor:
+    """``x`` fp32 [T, r] (rows may be strided), ``w2`` fp32 [C, r], ``bias`` fp32 [C] -> fp32 [T, C]. ``form`` "sigmoid":
+    sigmoid(w2 x + bias)^(1 / tau), formed as exp(log sigmoid(.) / tau); "exp_exp": exp(-exp(w2 tanh(x) + bias)). ``fast``: with the hardware's exponential and logarithm (models in 16 bits)."""
     T, r = x.shape
     C = w2.shape[0]
     if nv.use_native(x):
         if x.dtype != torch.float32 or x.stride(1) != 1:
             raise ValueError("lowrank_decay: fp32 rows with a contiguous last dim")
         out = torch.empty(T, C, dtype=torch.float32, device=x.device)
-        fn = nv.proto("b200_lowrank_decay", [vp, i64, vp, vp, vp, i32, i32, i32, f32, i32, vp])
-        nv.check(fn(nv.ptr(x), x.stride(0), nv.ptr(w2), nv.ptr(bias), nv.ptr(out), T, C, r, 1.0 / float(tau), int(fast), nv.stream()), "lowrank_decay")
+        fn = nv.proto("b200_lowrank_decay_ex", [vp, i64, vp, vp, vp, i32, i32, i32, f32, i32, i32, vp])
+        nv.check(fn(nv.ptr(x), x.stride(0), nv.ptr(w2), nv.ptr(bias), nv.ptr(out), T, C, r, 1.0 / float(tau), int(form == "exp_exp"), int(fast),
+                    nv.stream()), "lowrank_decay")
         nv.count_launch()
         return out
+    if form == "exp_exp":
+        return torch.exp(-torch.exp(torch.tanh(x.float()) @ w2.float().t() + bias.float()))
     z = x.float() @ w2.float().t() + bias.float()
     return torch.exp(F.logsigmoid(z) / tau)
 

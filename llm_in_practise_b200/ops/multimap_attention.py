@@ -7,8 +7,10 @@ can be combined differentially:
     o   = a_0 - lambda a_1;   o <- o / sqrt(mean(o^2) + eps) * post     (``combine``; M = 2)
 
 Keys live in ``cache_k`` [blocks, G * M, block, D] (after norm and rotation), values in ``cache_v`` [blocks, G, block, Dv];
-Dv need not equal D. A layer may attend over the pools another layer filled (shared K/V). ``qknorm_rope_store`` is the step
-in front: per-row RMS norm with a weight, split-half rotary on the first ``rot`` dims, the page writes. Beside
+Dv need not equal D. A layer may attend over the pools another layer filled (shared K/V). ``qkv_store`` (``qknorm_rope_store``)
+is the step in front: bias, per-row RMS norm with a weight, split-half rotary on the first ``rot`` dims, values mixed with
+another layer's, the page writes. One-map attention has options: capped scores, chunks instead of a window, a sink per head,
+a sigmoid gate per token and head. Beside
 ``ops.paged_attention`` (one map, values sized like keys, sinks) and ``ops.latent_attention`` (latent rows), which serve
 the same ragged step (the reference reaches it through vLLM, LLM_on_Kubernetes/Inference_Platfrom/README.md:1504-1509).
 """
@@ -24,9 +26,66 @@ from . import _native as nv
 from .linear_scan import _conv_tail, short_conv
 
 vp, i32, i64, f32 = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong, ctypes.c_float
-_MMA_D, _MMA_DV = (32, 48, 64, 96, 128), (32, 64, 96, 128)        # sizes the tensor-core kernel is built for
+_MMA_MAX = 128                                                     # largest key / value row of the tensor-core kernel
 _CONV_TAPS = 5                                                     # taps of the fused convolution + norm + store
 _SPLIT_KEYS = int(os.environ.get("B200_PAGED_SPLIT_KEYS", "512"))  # keys per range of a small batch with many visible keys
+
+
+class _AttnOpts(ctypes.Structure):
+    _fields_ = [("sink", vp), ("gate", vp), ("ld_gate", i64), ("softcap", f32), ("chunk", i32)]
+
+
+def qkv_store(proj: torch.Tensor, bias: Optional[torch.Tensor], wq: Optional[torch.Tensor], wk: Optional[torch.Tensor],
+              rope, pos: torch.Tensor, slot: torch.Tensor, cache_k: torch.Tensor, cache_v: torch.Tensor, table: torch.Tensor, H: int,
+              G: int, D: int, Dv: int, rot: int, eps: float, dtype: torch.dtype, v_first: Optional[torch.Tensor] = None,
+              v_lambda: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """What stands in front of one-map attention. ``proj`` [T, >= (H + G) D + G Dv] = q | k | v rows (fp32 or bf16) gets ``bias``
+    (fp32 [(H + G) D + G Dv] or None); q and k rows are RMS-normed with ``wq`` / ``wk`` (fp32 [D]; None: not normed) and their
+    first ``rot`` dims turned by the token's position (``rope`` = (cos, sin) fp32 [max_pos, rot / 2], split-half pairs; None
+    with ``rot`` 0). ``v_first``: the value pool of an earlier layer that already holds these tokens; then
+    v <- (1 - lambda) v + lambda v_first with ``v_lambda`` fp32 [1]. Returns q [T, H * D] in ``dtype``; keys and values are
+    written at (slot, pos) of the pools."""
+    T = proj.shape[0]
+    q_out = torch.empty(T, H * D, dtype=dtype, device=proj.device)
+    BS = cache_k.shape[2]
+    if v_first is not None and (v_first.shape != cache_v.shape or v_lambda is None):
+        raise ValueError("qkv_store: values can only be mixed with a pool of the same shape, by a lambda")
+    if nv.use_native(proj):
+        if proj.stride(1) != 1 or cache_k.dtype != dtype:
+            raise ValueError("qkv_store: rows with a contiguous last dim, q in the cache dtype")
+        cos, sin = rope if rope is not None else (None, None)
+        fn = nv.proto("b200_qkv_store", [vp, i64, vp, vp, vp, vp, vp, vp, vp, vp, i32, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32,
+                                         i32, i32, f32, i32, i32, i32, vp])
+        nv.check(fn(nv.ptr(proj), proj.stride(0), nv.ptr(bias), nv.ptr(wq), nv.ptr(wk), nv.ptr(cos), nv.ptr(sin), nv.ptr(pos), nv.ptr(slot),
+                    nv.ptr(table), table.shape[1], nv.ptr(q_out), nv.ptr(cache_k), nv.ptr(cache_v), nv.ptr(v_first), nv.ptr(v_lambda), T, H,
+                    G, 1, D, Dv, rot, BS, float(eps), 1, nv.dtype_code(proj.dtype), nv.dtype_code(dtype), nv.stream()), "qkv_store")
+        nv.count_launch()
+        return q_out
+    nq, nk = H * D, G * D
+    x = proj[:, :nq + nk + G * Dv].float()
+    if bias is not None:
+        x = x + bias.float()
+    pl, sl = pos.long(), slot.long()
+    hr = rot // 2
+
+    def prep(y, w):
+        if w is not None:
+            y = y * torch.rsqrt((y * y).mean(-1, keepdim=True) + eps) * w.float()
+        if rot:
+            c, s = rope[0][pl][:, None, :], rope[1][pl][:, None, :]
+            a, b = y[..., :hr], y[..., hr:rot]
+            y = torch.cat([a * c - b * s, b * c + a * s, y[..., rot:]], -1)
+        return y
+
+    q_out.copy_(prep(x[:, :nq].view(T, H, D), wq).reshape(T, nq).to(dtype))
+    blk, off = table[sl, pl // BS].long(), pl % BS
+    v = x[:, nq + nk:].reshape(T, G, Dv)
+    if v_first is not None:
+        lam = float(v_lambda)
+        v = (1.0 - lam) * v + lam * v_first[blk, :, off].float()
+    cache_k[blk, :, off] = prep(x[:, nq:nq + nk].view(T, G, D), wk).to(cache_k.dtype)
+    cache_v[blk, :, off] = v.to(cache_v.dtype)
+    return q_out
 
 
 def qknorm_rope_store(proj: torch.Tensor, wq: torch.Tensor, wk: Optional[torch.Tensor], cos: torch.Tensor, sin: torch.Tensor,
@@ -128,42 +187,59 @@ def conv_qknorm_store(proj: torch.Tensor, bias: Optional[torch.Tensor], w: torch
 def multimap_attention(q: torch.Tensor, cache_k: torch.Tensor, cache_v: torch.Tensor, table: torch.Tensor, pos: torch.Tensor,
                        slot: torch.Tensor, H: int, G: int, M: int, D: int, Dv: int, scale: float, window: int = 0,
                        keep_first: int = 0, combine: bool = False, lam: float = 0.0, post: float = 1.0, eps: float = 0.0,
-                       pieces=None, max_pos: int = 0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                       pieces=None, max_pos: int = 0, out: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None,
+                       softcap: float = 0.0, chunk: int = 0, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Context [T, H * Dv] (q's dtype) of ``q`` [T, H * M * D] over the pools; see the module docstring for the mask and the
     combination; ``post`` multiplies the result with and without it. ``out``: where to write it (rows may be strided). ``pieces`` (``inference.ragged.Pieces``): bf16 steps with a run of 8 or more tokens go through the tensor-core
     kernel; everything else (fp32, decode batches, sizes it is not built for) through the per-token kernels. ``max_pos``: an upper
-    bound of ``pos`` known on the host (0 = unknown), used to cut the keys of a small batch into ranges."""
+    bound of ``pos`` known on the host (0 = unknown), used to cut the keys of a small batch into ranges.
+
+    One-map options: ``softcap`` > 0: scores become c tanh(s / c); ``chunk`` > 0 (without a window): position p sees only keys
+    j <= p with j // chunk == p // chunk; ``sink`` fp32 [H]: exp(sink_h) joins the softmax's denominator; ``gate`` fp32 [T, H]
+    (rows may be strided): head h's output times sigmoid(gate[t, h])."""
     T = q.shape[0]
     BS = cache_k.shape[2]
     if out is None:
         out = torch.empty(T, H * Dv, dtype=q.dtype, device=q.device)
+    options = sink is not None or gate is not None or softcap or chunk
+    if options and (M != 1 or (chunk and window > 0)):
+        raise ValueError("multimap_attention: options are for one map, chunks for attention without a window")
     if nv.use_native(q):
+        opts = None
+        if options:
+            if (sink is not None and (sink.dtype != torch.float32 or sink.numel() != H)) or \
+                    (gate is not None and (gate.dtype != torch.float32 or gate.stride(1) != 1)):
+                raise ValueError("multimap_attention: sink fp32 [H], gate fp32 rows with a contiguous last dim")
+            opts = ctypes.byref(_AttnOpts(nv.ptr(sink), nv.ptr(gate), gate.stride(0) if gate is not None else 0, float(softcap), int(chunk)))
         if cache_k.dtype != q.dtype or not q.is_contiguous():
             raise ValueError("multimap_attention: contiguous q in the cache dtype")
         if out.dtype != q.dtype or out.stride(1) != 1:
             raise ValueError("multimap_attention: out in q's dtype with a contiguous last dim")
-        if (pieces is not None and pieces.longest >= 8 and q.dtype == torch.bfloat16 and D in _MMA_D and Dv in _MMA_DV and scale > 0
+        if (pieces is not None and pieces.longest >= 8 and q.dtype == torch.bfloat16 and D % 8 == 0 and Dv % 8 == 0
+                and max(D, Dv) <= _MMA_MAX and scale > 0
                 and BS & (BS - 1) == 0 and out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0 and os.environ.get("B200_PAGED_MMA", "1") != "0"):
-            fn = nv.proto("b200_multimap_attn_mma", [vp, vp, vp, vp, i32, vp, i32, vp, i64, i32, i32, i32, i32, i32, i32, f32, i32, i32, i32,
-                                                     f32, f32, f32, i32, vp])
+            fn = nv.proto("b200_multimap_attn_mma_ex", [vp, vp, vp, vp, i32, vp, i32, vp, i64, i32, i32, i32, i32, i32, i32, f32, i32, i32, i32,
+                                                        f32, f32, f32, vp, i32, vp])
             nv.check(fn(nv.ptr(q), nv.ptr(cache_k), nv.ptr(cache_v), nv.ptr(pieces.tiles), pieces.n_tiles, nv.ptr(table),
                         table.shape[1], nv.ptr(out), out.stride(0), H, G, M, D, Dv, BS, float(scale), int(window), int(keep_first), int(combine),
-                        float(lam), float(post), float(eps), nv.dtype_code(q.dtype), nv.stream()), "multimap_attn_mma")
+                        float(lam), float(post), float(eps), opts, nv.dtype_code(q.dtype), nv.stream()), "multimap_attn_mma")
             nv.count_launch()
             return out
         # few tokens with many visible keys (a small decode batch with a wide window or none): cut the keys into ranges
         seen = max_pos + 1 if max_pos > 0 else 0
         if window > 0:
             seen = min(seen, window + max(keep_first, 0))
+        if chunk > 0:
+            seen = min(seen, chunk)
         nsplit = 1
         if seen > 2 * _SPLIT_KEYS and T * G < 296:
             nsplit = min(32, -(-seen // _SPLIT_KEYS), max(1, 592 // (T * G)))
         part = torch.empty(T * H * M * nsplit * (Dv + 2), dtype=torch.float32, device=q.device) if nsplit * M > 1 else None
-        fn = nv.proto("b200_multimap_attn", [vp, vp, vp, vp, vp, vp, i32, vp, i64, vp, i32, i32, i32, i32, i32, i32, i32, f32, i32, i32,
-                                             i32, i32, f32, f32, f32, i32, vp])
+        fn = nv.proto("b200_multimap_attn_ex", [vp, vp, vp, vp, vp, vp, i32, vp, i64, vp, i32, i32, i32, i32, i32, i32, i32, f32, i32, i32,
+                                                i32, i32, f32, f32, f32, vp, i32, vp])
         nv.check(fn(nv.ptr(q), nv.ptr(cache_k), nv.ptr(cache_v), nv.ptr(pos), nv.ptr(slot), nv.ptr(table), table.shape[1],
                     nv.ptr(out), out.stride(0), nv.ptr(part), T, H, G, M, D, Dv, BS, float(scale), int(window), int(keep_first), nsplit, int(combine),
-                    float(lam), float(post), float(eps), nv.dtype_code(q.dtype), nv.stream()), "multimap_attn")
+                    float(lam), float(post), float(eps), opts, nv.dtype_code(q.dtype), nv.stream()), "multimap_attn")
         nv.count_launch(2 if nsplit * M > 1 else 1)
         return out
     rep = H // G
@@ -171,18 +247,24 @@ def multimap_attention(q: torch.Tensor, cache_k: torch.Tensor, cache_v: torch.Te
     qf = q.float().view(T, H, M, D)
     for t in range(T):
         p = pl[t]
-        lo = max(0, p + 1 - window) if window > 0 else 0
-        idx = list(range(min(max(keep_first, 0), lo))) + list(range(lo, p + 1))
+        lo = max(0, p + 1 - window) if window > 0 else (p // chunk * chunk if chunk else 0)
+        idx = list(range(min(max(keep_first, 0), lo) if window > 0 else 0)) + list(range(lo, p + 1))
         it = torch.tensor(idx, dtype=torch.long, device=q.device)
         blk = table[sl[t], it // BS].long()
         off = it % BS
         k = cache_k[blk, :, off].float().view(len(idx), G, M, D).repeat_interleave(rep, 1)        # [n, H, M, D]
         v = cache_v[blk, :, off].float().repeat_interleave(rep, 1)                                 # [n, H, Dv]
         sc = torch.einsum("hmd,nhmd->hmn", qf[t], k) * scale
-        a = torch.einsum("hmn,nhe->hme", sc.softmax(-1), v)
+        if softcap:
+            sc = softcap * torch.tanh(sc / softcap)
+        if sink is not None:
+            sc = torch.cat([sc, sink.float().view(H, 1, 1)], -1)
+        a = torch.einsum("hmn,nhe->hme", sc.softmax(-1)[:, :, :len(idx)], v)
         o = a[:, 0] - lam * a[:, 1] if M == 2 else a[:, 0]
         if combine:
             o = o * torch.rsqrt((o * o).mean(-1, keepdim=True) + eps)
         o = o * post
+        if gate is not None:
+            o = o * torch.sigmoid(gate[t].float())[:, None]
         out[t] = o.reshape(H * Dv).to(q.dtype)
     return out

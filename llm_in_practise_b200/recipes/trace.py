@@ -29,6 +29,8 @@ NATIVE_SOURCES = {
                 "talking_attn_mma"],
     "Lorenex": ["gemm_tcgen05", "gemv", "gemm_simt", "norm", "elementwise", "moe", "linear_scan", "channel_scan", "selective_scan",
                 "multimap_attn", "multimap_attn_mma"],
+    "Nedesun": ["gemm_tcgen05", "gemv", "gemm_simt", "norm", "elementwise", "linear_scan", "channel_scan", "multimap_attn",
+                "multimap_attn_mma"],
 }
 BLOCK = 64
 MAX_LIVE = 4
