@@ -46,10 +46,10 @@ def parse_args():
     ap.add_argument("--sequential-accum", action="store_true",
                     help="run the micro-batches one after the other (the earlier schedule) instead of one layer-major pass")
     ap.add_argument("--local_rank", type=int, default=-1)
-    ap.add_argument("--workload", default="headline", choices=["headline", "gorozen", "segorax", "duratar", "kudonex", "lorenex"],
+    ap.add_argument("--workload", default="headline", choices=["headline", "gorozen", "segorax", "duratar", "kudonex", "lorenex", "nedesun"],
                     help="gorozen: prefill / decode throughput and kernel rooflines of the Gorozen design beside Qwen3 at equal "
                          "layer sizes (one GPU, serving path); segorax / duratar: the same for those designs beside Gorozen; "
-                         "kudonex: the same beside Duratar; lorenex: the same beside Kudonex; the default is the headline training step")
+                         "kudonex: the same beside Duratar; lorenex: the same beside Kudonex; nedesun: the same beside Lorenex; the default is the headline training step")
     return ap.parse_args()
 
 
@@ -151,6 +151,10 @@ def main():
         sys.path.insert(0, os.path.join(ROOT, "bench"))
         import lorenex_bench
         return lorenex_bench.run(args, ROOT)
+    if args.workload == "nedesun":
+        sys.path.insert(0, os.path.join(ROOT, "bench"))
+        import nedesun_bench
+        return nedesun_bench.run(args, ROOT)
 
     import torch
     import torch.distributed as dist
