@@ -48,8 +48,9 @@ struct ChannelScanArgs {
 };
 
 // PASS 0: blockIdx.x is a run; 1, 2: a tile
+// Four CTAs per SM for short runs and decode batches (0: the compiler's own choice; the tile passes are faster with it).
 template <int PASS, int LPC, bool BONUS>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, PASS == 0 ? 4 : 0)
 channel_scan_kernel(const ChannelScanArgs a) {
   extern __shared__ __align__(16) float sm[];
   constexpr int R = kCsR, CPT = kCsCols, RP = R + 4, DP = LPC * RP, cpw = 32 / LPC;
@@ -124,14 +125,16 @@ channel_scan_kernel(const ChannelScanArgs a) {
 #pragma unroll
   for (int i = 0; i < R / 2; ++i) P2[i] = make_float2(1.f, 1.f);
 
+  // the bonus of a thread's rows stays in registers over a tile; a short run reads it per token instead (occupancy)
   float2 u2[R / 2];
-  if (BONUS && PASS != 1) {
+  auto load_u = [&]() {
 #pragma unroll
     for (int i = 0; i < R / 2; ++i) {
-      u2[i].x = row0 + 2 * i < D ? a.u[h * D + row0 + 2 * i] : 0.f;
-      u2[i].y = row0 + 2 * i + 1 < D ? a.u[h * D + row0 + 2 * i + 1] : 0.f;
+      u2[i].x = row0 + 2 * i < D ? __ldg(a.u + h * D + row0 + 2 * i) : 0.f;
+      u2[i].y = row0 + 2 * i + 1 < D ? __ldg(a.u + h * D + row0 + 2 * i + 1) : 0.f;
     }
-  }
+  };
+  if (BONUS && PASS == 2) load_u();
 
   auto stage = [&](int b, int c0) {
     const int cn = min(CH, n - c0);
@@ -199,6 +202,7 @@ channel_scan_kernel(const ChannelScanArgs a) {
       float o[CPT];
       float bonus = 0.f;                                 // this lane's part of q . diag(u) k, the weight of the token's own value
       if (BONUS && PASS != 1) {
+        if (PASS == 0) load_u();
         float2 ba = make_float2(0.f, 0.f);
 #pragma unroll
         for (int i = 0; i < R / 2; ++i) ba = __ffma2_rn(__fmul2_rn(u2[i], k2[i]), q2[i], ba);

@@ -212,9 +212,18 @@ delta_gates_kernel(float* __restrict__ q, long long ldq, float* __restrict__ k, 
                    const float* __restrict__ A_log, int G, int H, int D, int AD, float qscale, float unit_eps) {
   const int t = blockIdx.x;                               // AD: decays per head (D, or 1)
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-  for (int r = warp; r < 2 * G + H; r += nw) {
+  const bool v4 = D % 4 == 0 && D <= 128 && ldq % 4 == 0 && ldk % 4 == 0 &&
+                  !((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k)) & 15);
+  for (int r = warp; r < 2 * G + (AD > 1 ? H : 0); r += nw) {
     if (r < 2 * G) {
       float* x = r < G ? q + (long long)t * ldq + (long long)r * D : k + (long long)t * ldk + (long long)(r - G) * D;
+      if (v4) {                                           // a row is at most one 16-byte group per lane
+        float4 u = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (lane * 4 < D) u = *reinterpret_cast<const float4*>(x + lane * 4);
+        const float sc = rsqrtf(warp_sum(u.x * u.x + u.y * u.y + u.z * u.z + u.w * u.w) + unit_eps) * (r < G ? qscale : 1.f);
+        if (lane * 4 < D) *reinterpret_cast<float4*>(x + lane * 4) = make_float4(u.x * sc, u.y * sc, u.z * sc, u.w * sc);
+        continue;
+      }
       float ss = 0.f;
       for (int d = lane; d < D; d += 32) ss += x[d] * x[d];
       ss = warp_sum(ss);
@@ -234,6 +243,11 @@ delta_gates_kernel(float* __restrict__ q, long long ldq, float* __restrict__ k, 
   for (int h = threadIdx.x; h < H; h += blockDim.x) {
     float* x = b + (long long)t * ldb + h;
     *x = 1.f / (1.f + expf(-*x));
+    if (AD == 1) {
+      float* y = a + (long long)t * lda + h;
+      const float z = *y + dt_bias[h];
+      *y = expf(-expf(A_log[h]) * (z > 20.f ? z : log1pf(expf(z))));
+    }
   }
 }
 

@@ -29,7 +29,8 @@ __device__ __forceinline__ float tanh_series(float x) {
   return x * fmaf(y, fmaf(y, fmaf(y, fmaf(y, 62.f / 2835.f, -17.f / 315.f), 2.f / 15.f), -1.f / 3.f), 1.f);
 }
 
-template <int DK, int DVK>
+// CAP: capped scores or chunks (the plain instance keeps their tests out of the loop)
+template <int DK, int DVK, bool CAP>
 __global__ void __launch_bounds__(128)
 multimap_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ ck,
                          const __nv_bfloat16* __restrict__ cv, const int* __restrict__ tiles, const int* __restrict__ table,
@@ -50,7 +51,7 @@ multimap_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
   const int nkb = (kv_len + kK - 1) / kK;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int bs_mask = (1 << bs_log2) - 1;
-  const int chunk = opt.chunk;
+  const int chunk = CAP ? opt.chunk : 0;
   // the first key a row sees besides kept ones: the window's lower edge, or the start of its chunk
   auto low_of = [&](int p) { return chunk > 0 ? p / chunk * chunk : (window > 0 ? max(0, p + 1 - window) : 0); };
   const int lo0 = low_of(pos0);
@@ -65,7 +66,7 @@ multimap_attn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
   for (int i = 0; i < 2 * DVK; ++i) res[i][0] = res[i][1] = res[i][2] = res[i][3] = 0.f;
   const int qpos0 = pos0 + warp * 16 + (lane >> 2);       // position of this thread's first row; the second is + 8
   const float LOG2E = 1.4426950408889634f;
-  const bool capped = opt.softcap > 0.f;
+  const bool capped = CAP && opt.softcap > 0.f;
   const float sl2 = capped ? opt.softcap * LOG2E : scale * LOG2E;        // capped: scores become tanh(q . k scale / cap) first
   const float cin = capped ? scale / opt.softcap : 0.f;
   const int low_a = low_of(qpos0), low_b = low_of(qpos0 + 8), low_w = low_of(pos0 + warp * 16 + 15);
@@ -281,7 +282,7 @@ static int launch(const void* q, const void* ck, const void* cv, const int* tile
                   int combine, float lambda, float post, float eps, const b200_attn_opts& opt, cudaStream_t st) {
   constexpr int LDK = 16 * DK + 8, LDV = 16 * DVK + 8;
   const size_t smem = ((size_t)(kQ + 2 * kK) * LDK + (size_t)2 * kK * LDV) * sizeof(__nv_bfloat16);
-  auto kern = multimap_attn_mma_kernel<DK, DVK>;
+  auto kern = opt.softcap > 0.f || opt.chunk > 0 ? multimap_attn_mma_kernel<DK, DVK, true> : multimap_attn_mma_kernel<DK, DVK, false>;
   if (smem > 48 * 1024) B200_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   int bs_log2 = 0;
   while ((1 << bs_log2) < block_size) ++bs_log2;

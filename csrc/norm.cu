@@ -500,9 +500,109 @@ sandwich_norm_kernel(const TY* __restrict__ y, const WT* __restrict__ w_post, co
     h[row * cols + i] = from_f32<TH>((rowbuf[i] - m2) * r2 * (off + to_f32<WT>(w_next[i])));
 }
 
+// four neighbouring elements as fp32, and back
+template <typename T> __device__ __forceinline__ float4 load4(const T* p) {
+  if constexpr (sizeof(T) == 4) {
+    return *reinterpret_cast<const float4*>(p);
+  } else {
+    const uint2 r = *reinterpret_cast<const uint2*>(p);
+    const T* e = reinterpret_cast<const T*>(&r);
+    return make_float4(to_f32<T>(e[0]), to_f32<T>(e[1]), to_f32<T>(e[2]), to_f32<T>(e[3]));
+  }
+}
+template <typename T> __device__ __forceinline__ void store4(T* p, const float4 v) {
+  if constexpr (sizeof(T) == 4) {
+    *reinterpret_cast<float4*>(p) = v;
+  } else {
+    uint2 r;
+    T* e = reinterpret_cast<T*>(&r);
+    e[0] = from_f32<T>(v.x); e[1] = from_f32<T>(v.y); e[2] = from_f32<T>(v.z); e[3] = from_f32<T>(v.w);
+    *reinterpret_cast<uint2*>(p) = r;
+  }
+}
+__device__ __forceinline__ float dot4(const float4 v) { return fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w))); }
+
+// The RMS case of the kernel above for rows of whole groups of four columns: a thread keeps its NV groups in registers from the
+// first load to the last store, so nothing passes through shared memory but the sums.
+template <typename TY, typename TH, typename WT, int NV, bool TWO>
+__global__ void __launch_bounds__(kNormThreads)
+sandwich_norm_vec_kernel(const TY* __restrict__ y, const WT* __restrict__ w_post, const TY* __restrict__ y2,
+                         const WT* __restrict__ w_post2, const float* __restrict__ res_in, float* __restrict__ res_out,
+                         const WT* __restrict__ w_next, TH* __restrict__ h, int cols, float eps, float off, float mult) {
+  __shared__ float red[32];
+  const long long base = (long long)blockIdx.x * cols;
+  float4 v[NV], v2[NV], x[NV];
+  float ss = 0.f, s3 = 0.f;
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int i = (threadIdx.x + j * blockDim.x) * 4;
+    v[j] = v2[j] = x[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i >= cols) continue;
+    if (y) v[j] = load4<TY>(y + base + i);
+    if (TWO) v2[j] = load4<TY>(y2 + base + i);
+    if (res_in) x[j] = *reinterpret_cast<const float4*>(res_in + base + i);
+  }
+  float r1 = 1.f, r3 = 1.f;
+  if (w_post) {
+#pragma unroll
+    for (int j = 0; j < NV; ++j) { ss += dot4(v[j]); if (TWO) s3 += dot4(v2[j]); }
+    r1 = 1.f / sqrtf(block_sum(ss, red) / (float)cols + eps);
+    if (TWO) r3 = 1.f / sqrtf(block_sum(s3, red) / (float)cols + eps);
+  }
+  float s2 = 0.f;
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int i = (threadIdx.x + j * blockDim.x) * 4;
+    if (i >= cols) continue;
+    if (w_post) {
+      const float4 w = load4<WT>(w_post + i);
+      v[j] = make_float4(v[j].x * r1 * (off + w.x), v[j].y * r1 * (off + w.y), v[j].z * r1 * (off + w.z), v[j].w * r1 * (off + w.w));
+    }
+    if (TWO) {
+      const float4 w = load4<WT>(w_post2 + i);
+      v[j] = make_float4(fmaf(v2[j].x * r3, off + w.x, v[j].x), fmaf(v2[j].y * r3, off + w.y, v[j].y), fmaf(v2[j].z * r3, off + w.z, v[j].z),
+                         fmaf(v2[j].w * r3, off + w.w, v[j].w));
+    }
+    x[j] = make_float4(fmaf(v[j].x, mult, x[j].x), fmaf(v[j].y, mult, x[j].y), fmaf(v[j].z, mult, x[j].z), fmaf(v[j].w, mult, x[j].w));
+    if (res_out) *reinterpret_cast<float4*>(res_out + base + i) = x[j];
+    s2 += dot4(x[j]);
+  }
+  float r2 = 1.f;
+  if (w_next) r2 = 1.f / sqrtf(block_sum(s2, red) / (float)cols + eps);
+  if (!h) return;
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int i = (threadIdx.x + j * blockDim.x) * 4;
+    if (i >= cols) continue;
+    if (w_next) {
+      const float4 w = load4<WT>(w_next + i);
+      x[j] = make_float4(x[j].x * r2 * (off + w.x), x[j].y * r2 * (off + w.y), x[j].z * r2 * (off + w.z), x[j].w * r2 * (off + w.w));
+    }
+    store4<TH>(h + base + i, x[j]);
+  }
+}
+
 template <typename TY, typename TH, typename WT>
 static int sandwich_launch(const void* y, const void* w_post, const void* y2, const void* w_post2, const float* res_in, float* res_out,
                            const void* w_next, void* h, long long rows, int cols, float eps, float off, float mult, int center, cudaStream_t st) {
+  {
+    auto al = [](const void* p_, size_t es) { return !(reinterpret_cast<uintptr_t>(p_) & (4 * es - 1)); };
+    if (!center && cols % 4 == 0 && cols <= 16 * kNormThreads * 2 && al(y, sizeof(TY)) && al(y2, sizeof(TY)) && al(w_post, sizeof(WT)) &&
+        al(w_post2, sizeof(WT)) && al(w_next, sizeof(WT)) && al(res_in, 4) && al(res_out, 4) && al(h, sizeof(TH))) {
+      const int groups = (cols / 4 + kNormThreads - 1) / kNormThreads;
+      int nt = (cols / 4 + groups - 1) / groups;          // no more threads than groups of columns
+      nt = nt > kNormThreads ? kNormThreads : (nt + 31) / 32 * 32;
+#define SWV(NV, TWO)                                                                                                          \
+  sandwich_norm_vec_kernel<TY, TH, WT, NV, TWO><<<(unsigned)rows, nt, 0, st>>>((const TY*)y, (const WT*)w_post, (const TY*)y2,  \
+      (const WT*)w_post2, res_in, res_out, (const WT*)w_next, (TH*)h, cols, eps, off, mult)
+#define SWV_N(NV) do { if (y2) SWV(NV, true); else SWV(NV, false); } while (0)
+      if (groups <= 1) SWV_N(1); else if (groups <= 2) SWV_N(2); else if (groups <= 4) SWV_N(4); else SWV_N(8);
+#undef SWV_N
+#undef SWV
+      B200_LAUNCH_CHECK();
+      return 0;
+    }
+  }
   const size_t smem = (size_t)cols * (y2 ? 2 : 1) * sizeof(float);
   auto kern = sandwich_norm_kernel<TY, TH, WT>;
   if (smem > 48 * 1024) {
