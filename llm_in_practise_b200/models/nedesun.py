@@ -226,7 +226,7 @@ class NedesunLayer(nn.Module):
         lo, hi = self.parts[name]
         return main[:, lo:hi] if hi <= self.main else tail[:, lo - self.main:hi - self.main]
 
-    # ------------------------------------------------------------------ mixers: h [T, W] (model dtype) -> fp32 [T, W]
+    # ------------------------------------------------------------------ mixers: h [T, W] (model dtype) -> fp32 [T, W] (parallel: one per half)
     def parallel(self, h, pos, slot, state, cache, li: int, pieces, eps: float, max_pos: int):
         m = self.spec.mixer
         dt = h.dtype
